@@ -8,7 +8,11 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libbpdq.so")
-SOURCES = ["runtime.cu", "dequant_q4k.cu", "gemv_q4k.cu", "gemv_batch.cu", "gemv_persistent.cu", "gemv_stream.cu", "q8_0.cu", "w4a32.cu", "decode_ops.cu", "gemm_q4k_mma.cu", "gemm_q4k_tc5.cu", "gemm_q4k_rg16.cu", "gemm_q8_0_tiles.cu", "llama_forward.cu", "peer_exchange.cu"]
+SOURCES = ["runtime.cu", "dequant_q4k.cu", "gemv_q4k.cu", "gemv_batch.cu", "gemv_persistent.cu", "gemv_stream.cu", "q8_0.cu", "w4a32.cu", "decode_ops.cu", "gemm_q4k_mma.cu", "gemm_q4k_tc5.cu", "gemm_q4k_rg16.cu", "gemm_q8_0_tiles.cu", "llama_forward.cu", "peer_exchange.cu",
+           "linear.cu", "decayed_scan.cu", "latent_attention.cu", "hybrid_forward.cu"]
+# The sources one model family needs: a process that only serves that family (bin/trace_run in a fresh checkout)
+# compiles and loads these as a library of their own when the whole one has not been built.
+PARTS = {"hybrid": ["runtime.cu", "decode_ops.cu", "linear.cu", "decayed_scan.cu", "latent_attention.cu", "hybrid_forward.cu"]}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
@@ -22,24 +26,29 @@ def _nvcc():
     raise RuntimeError("nvcc not found: libbpdq.so cannot be built")
 
 
-def _stale():
-    if not os.path.exists(LIB):
+def lib_path(part=None):
+    return LIB if part is None else os.path.join(HERE, f"libbpdq_{part}.so")
+
+
+def _stale(lib):
+    if not os.path.exists(lib):
         return True
-    t = os.path.getmtime(LIB)
+    t = os.path.getmtime(lib)
     deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)]
     deps.append(os.path.join(HERE, "..", "include", "bpdq.h"))
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force=False, verbose=False):
-    """Compile every .cu to an object (in parallel) and link libbpdq.so."""
-    if not force and not _stale():
-        return LIB
+def build(force=False, verbose=False, part=None):
+    """Compile every .cu (of a part) to an object, in parallel, and link libbpdq.so (libbpdq_<part>.so)."""
+    lib = lib_path(part)
+    if not force and not _stale(lib):
+        return lib
     nvcc = _nvcc()
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
     procs = []
-    for src in SOURCES:
+    for src in SOURCES if part is None else PARTS[part]:
         obj = os.path.join(objdir, src.replace(".cu", ".o"))
         cmd = [nvcc, *NVCC_FLAGS, *os.environ.get("BPDQ_NVCC_FLAGS", "").split(), "-c", os.path.join(CSRC, src), "-o", obj]
         if verbose:
@@ -53,8 +62,10 @@ def build(force=False, verbose=False):
         if p.returncode:
             raise RuntimeError(f"nvcc failed on {src}")
         objs.append(obj)
-    subprocess.check_call([nvcc, "-shared", "-o", LIB, *objs, "-gencode", "arch=compute_100a,code=sm_100a"])
-    return LIB
+    tmp = f"{lib}.{os.getpid()}"
+    subprocess.check_call([nvcc, "-shared", "-o", tmp, *objs, "-gencode", "arch=compute_100a,code=sm_100a"])
+    os.replace(tmp, lib)
+    return lib
 
 
 if __name__ == "__main__":

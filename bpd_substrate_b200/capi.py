@@ -168,6 +168,20 @@ SIGNATURES = {
     "bpd_unrepack_q8_0_tiles_cuda": (i32, [vp, vp, i32, i32, vp]),
     "bpd_qmatmul_q8_0_tiles_cuda": (i32, [vp, vp, vp, i32, i32, i32, vp]),
     "gpu_vecmat_q8_0": (None, [vp, vp, vp, i32, i32]),
+    # hybrid decoder
+    "bpd_linear_bf16_cuda": (i32, [vp, vp, vp, i32, i32, i32, i32, vp]),
+    "bpd_decayed_scan_cuda": (i32, [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]),
+    "bpd_rotate_half_qk_cuda": (i32, [vp, vp, i32, i32, i32, i32, i32, vp, f32, vp, i32, vp]),
+    "bpd_causal_conv_silu_cuda": (i32, [vp, i32, vp, i32, i32, i32, vp, vp, vp, i32, vp]),
+    "bpd_gated_norm_cuda": (i32, [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp]),
+    "bpd_latent_prepare_cuda": (i32, [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, vp]),
+    "bpd_latent_attention_cuda": (i32, [vp, vp, vp, vp, vp, vp, i32, i32, i32, vp]),
+    "bpdq_hybrid_create": (vp, [vp, vp]),
+    "bpdq_hybrid_destroy": (None, [vp]),
+    "bpdq_hybrid_forward": (i32, [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp]),
+    "bpdq_hybrid_logits": (vp, [vp]),
+    "bpdq_hybrid_picked": (vp, [vp]),
+    "bpdq_hybrid_scratch_bytes": (sz, [vp]),
     "gpu_matmul_q4k": (None, [vp, vp, vp, i32, i32, i32]),
 }
 
@@ -176,18 +190,25 @@ def lib_path():
     return _build.LIB
 
 
-def load(build_if_missing=True):
-    """Returns the bound library; raises if it cannot be built or loaded."""
+def load(build_if_missing=True, part=None):
+    """Returns the bound library; raises if it cannot be built or loaded.  part: a process that only needs one model
+    family's entries may load that family's library instead when the whole one has not been built."""
     global _LIB
     if _LIB is not None:
         return _LIB
     path = lib_path()
+    if part is not None and not os.path.exists(path):
+        path = _build.build(part=part) if build_if_missing else _build.lib_path(part)
+    else:
+        part = None
     if not os.path.exists(path):
         if not build_if_missing:
             raise FileNotFoundError(f"{path} is missing: run bpd_substrate_b200._build.build()")
         _build.build()
     lib = C.CDLL(path)
     for name, (res, args) in SIGNATURES.items():
+        if part is not None and not hasattr(lib, name):
+            continue
         fn = getattr(lib, name)   # AttributeError if the symbol is not exported
         fn.restype = res
         fn.argtypes = args
@@ -222,6 +243,37 @@ class LlamaWeights(C.Structure):
     """bpd_llama_weights; `layers` points to a host array of LlamaLayerWeights."""
     _fields_ = [("token_embd", vp), ("layers", C.POINTER(LlamaLayerWeights)), ("output_norm_w", vp), ("output_w", vp),
                 ("rope_freqs", vp)]
+
+
+class LatentShape(C.Structure):
+    """bpdq_latent_shape."""
+    _fields_ = [(n, i32) for n in ("heads", "dim_pad", "value_pad", "rank", "rank_pad", "rot_dims", "rot_pad", "q_rank",
+                                   "q_rank_pad")] + [("scale", f32), ("eps", f32), ("rot_freq", vp)]
+
+
+class DynTanh(C.Structure):
+    """bpdq_dyn_tanh."""
+    _fields_ = [("w", vp), ("b", vp), ("alpha", f32)]
+
+
+MIX_RETENTION, MIX_MAMBA2, MIX_LATENT = 0, 1, 2
+
+
+class HybridLayer(C.Structure):
+    """bpdq_hybrid_layer."""
+    _fields_ = ([(n, i32) for n in ("mixer", "heads", "groups", "key_dim", "key_pad", "value_dim", "value_pad", "rot_dims", "rot_pad",
+                                    "conv", "norm_groups", "q_rank", "q_rank_pad", "kv_rank", "kv_rank_pad", "kv_from", "ff_pad")]
+                + [("scale", f32)]
+                + [(n, vp) for n in ("rot_freq", "decay", "log_decay", "conv_w", "conv_b", "dt_bias", "neg_exp_a", "d_skip", "norm_w",
+                                     "q_norm_w", "kv_norm_w", "w_in", "w_uq", "w_ukv", "w_o", "w_gate_up", "w_down")]
+                + [(n, DynTanh) for n in ("norm1", "norm1b", "norm2", "norm2b")]
+                + [(n, sz) for n in ("state_offset", "tail_offset", "cache_offset")])
+
+
+class HybridConfig(C.Structure):
+    """bpdq_hybrid_config."""
+    _fields_ = [(n, i32) for n in ("n_layers", "width", "width_pad", "vocab", "act_bf16")] + [("eps", f32), ("embed", vp),
+                                                                                              ("final_norm", DynTanh)]
 
 
 class BpdqError(RuntimeError):

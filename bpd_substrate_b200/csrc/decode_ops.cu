@@ -4,6 +4,7 @@
 // :600-830, k_matmul :1104-1290).  They sit either side of the quantized GEMVs in a decode
 // step; all are memory bound and small.
 #include "bpdq_common.cuh"
+#include "launch.cuh"
 #include "../../include/bpdq.h"
 
 namespace bpdq {
@@ -95,6 +96,37 @@ __global__ void __launch_bounds__(1024) k_matmul_f32(const float* __restrict__ A
     if (row < M && col < N) C[(size_t)row * N + col] = acc;
 }
 
+// One CTA per row; the largest value wins, the lowest index among equals (v > best in index order).
+__global__ void __launch_bounds__(256) k_argmax_rows(const float* x, long long* out, int n)
+{
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float s_v[256];
+    __shared__ int s_i[256];
+    const float* row = x + (size_t)blockIdx.x * n;
+    float best = row[0];
+    int bi = 0;
+    for (int k = threadIdx.x; k < n; k += 256) {
+        const float v = row[k];
+        if (v > best || (v == best && k < bi)) { best = v; bi = k; }
+    }
+    s_v[threadIdx.x] = best;
+    s_i[threadIdx.x] = bi;
+    __syncthreads();
+    for (int o = 128; o > 0; o >>= 1) {
+        if (threadIdx.x < o) {
+            const float v = s_v[threadIdx.x + o];
+            const int i = s_i[threadIdx.x + o];
+            if (v > s_v[threadIdx.x] || (v == s_v[threadIdx.x] && i < s_i[threadIdx.x])) {
+                s_v[threadIdx.x] = v;
+                s_i[threadIdx.x] = i;
+            }
+        }
+        __syncthreads();
+    }
+    if (threadIdx.x == 0) out[blockIdx.x] = s_i[0];
+}
+
 static int ew_grid(long n)
 {
     long want = (n + 255) / 256, cap = (long)sm_count() * 8;
@@ -150,5 +182,14 @@ void gpu_matmul(const float* A, const float* B, float* C, int M, int N, int K)
     check_cuda(cudaGetLastError());
 }
 void gpu_matmul_opt(const float* A, const float* B, float* C, int M, int N, int K) { gpu_matmul(A, B, C, M, N, K); }
+
+int bpd_argmax_dim_cuda(const float* x, long long* out, int outer, int dim_size, int inner, void* stream)
+{
+    if (outer < 0 || dim_size < 1 || inner != 1 || (outer > 0 && (!x || !out))) return latch(BPDQ_ERR_ARG);
+    if (outer == 0) return 0;
+    launch_ordered(k_argmax_rows, outer, 256, 0, (cudaStream_t)stream, x, out, dim_size);
+    int rc = check_cuda(cudaGetLastError());
+    return rc ? latch(rc) : 0;
+}
 
 }  // extern "C"

@@ -1,0 +1,128 @@
+// Building blocks shared by the kernels of the hybrid decoder (recurrent and latent-attention layers on bf16
+// weights): activation types, the dynamic-tanh norm, the epilogues of its matrix products, bf16 tensor-core
+// fragments.
+//
+// Weights are bf16.  Activations are bf16 or fp32 (the template parameter A); the residual stream, norms, scores,
+// softmax, decays and recurrent states are fp32 in both cases.  Every inner size is padded to a multiple of 16 with
+// zero weights when a model is loaded, so rows are 16-byte aligned and kernels need no ragged inner loops; pad
+// columns of activations hold finite values that meet zero weights.
+#pragma once
+#include "bpdq_common.cuh"
+
+#include <cuda_bf16.h>
+
+namespace bpdq {
+
+typedef __nv_bfloat16 bf16;
+
+// tanh(alpha x) * w + b, element by element (no statistics).  w == null: no norm.
+struct DynTanh {
+    const float *w, *b;
+    float alpha;
+};
+
+enum LinearMode {
+    kLinAct = 0,        // out[t][n] = A(v)
+    kLinF32 = 1,        // out[t][n] = v
+    kLinResidual = 2,   // x[t][n] += post(v); out[t][n] = A(next(x[t][n])) when `next` is given
+    kLinSwiglu = 3,     // rows come in pairs (2i: gate, 2i + 1: up); out[t][i] = A(silu(gate) * up)
+    kLinSsmIn = 4       // rows >= dt_row are step sizes: dt[t][n - dt_row] = softplus(v + dt_bias) in fp32; with
+                        // conv.w also the rows of [conv_row, dt_row) pass the causal convolution (one token only)
+};
+
+// Depthwise causal convolution of one token: tail [taps - 1][channels] holds the inputs before it, oldest first.
+struct ConvStep {
+    const float *w, *b;     // w [taps][channels]; w == null: no convolution here
+    float* tail;
+    void* out;              // [channels], activation type
+    int taps, channels;
+};
+
+struct Linear {
+    const bf16* W;          // [N][K]
+    const void* in;         // [T][ld_in], activation type
+    int N, K, ld_in;
+    int mode;
+    void* out;
+    int ld_out;
+    float* x;               // residual stream [T][ld_x]
+    int ld_x;
+    DynTanh post, next;
+    int conv_row, dt_row;
+    const float* dt_bias;
+    float* dt;              // [T][ld_dt]
+    int ld_dt;
+    ConvStep conv;
+};
+
+// Runs one product over T tokens (linear.cu); act_bf16: A is bf16, else fp32.
+int linear_forward(const Linear& l, int T, bool act_bf16, cudaStream_t s);
+
+#ifdef __CUDACC__
+
+template <typename A> __device__ __forceinline__ float act_load(const A* p);
+template <> __device__ __forceinline__ float act_load<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float act_load<bf16>(const bf16* p) { return __bfloat162float(*p); }
+template <typename A> __device__ __forceinline__ A act_from(float v);
+template <> __device__ __forceinline__ float act_from<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 act_from<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+template <typename A> __device__ __forceinline__ float act_round(float v);
+template <> __device__ __forceinline__ float act_round<float>(float v) { return v; }
+template <> __device__ __forceinline__ float act_round<bf16>(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
+
+// Four consecutive activations (16-byte or 8-byte aligned).
+__device__ __forceinline__ float4 act_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 act_load4(const bf16* p)
+{
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xFFFF0000u));
+}
+
+__device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float dyn_tanh(const DynTanh& p, int n, float v) { return fmaf(tanhf(p.alpha * v), p.w[n], p.b[n]); }
+
+// Everything but the pairwise mode: row n, token t.
+template <typename A>
+__device__ __forceinline__ void linear_store(const Linear& l, int t, int n, float v)
+{
+    switch (l.mode) {
+    case kLinF32: reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n] = v; break;
+    case kLinResidual: {
+        float* px = l.x + (size_t)t * l.ld_x + n;
+        const float r = *px + dyn_tanh(l.post, n, v);
+        *px = r;
+        if (l.next.w) reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(dyn_tanh(l.next, n, r));
+        break;
+    }
+    case kLinSsmIn:
+        if (n >= l.dt_row) {
+            l.dt[(size_t)t * l.ld_dt + n - l.dt_row] = softplus_f32(v + l.dt_bias[n - l.dt_row]);
+            break;
+        }
+        if (l.conv.w && n >= l.conv_row) {
+            const int c = n - l.conv_row, C = l.conv.channels;
+            float acc = l.conv.b[c];
+            for (int j = 0; j + 1 < l.conv.taps; j++) {
+                const float u = l.conv.tail[(size_t)j * C + c];
+                acc = fmaf(l.conv.w[(size_t)j * C + c], u, acc);
+                if (j > 0) l.conv.tail[(size_t)(j - 1) * C + c] = u;
+            }
+            // the window holds activations: in bf16 runs the newest input is rounded as a prompt's projection is
+            const float u = act_round<A>(v);
+            const int last = l.conv.taps - 1;
+            acc = fmaf(l.conv.w[(size_t)last * C + c], u, acc);
+            if (last > 0) l.conv.tail[(size_t)(last - 1) * C + c] = u;
+            reinterpret_cast<A*>(l.conv.out)[c] = act_from<A>(silu_f32(acc));
+            break;
+        }
+        reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(v);
+        break;
+    default: reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(v);
+    }
+}
+
+#endif
+}  // namespace bpdq

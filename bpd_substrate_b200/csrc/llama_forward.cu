@@ -5,7 +5,8 @@
 //   rotary embedding, NORM pairing, freq factors   bench/bpd_cpu.c:5146-5183
 //   f16 KV-cache write (round to nearest even)     bench/bpd_cpu.c:5240-5257
 //   grouped-query attention, three-pass softmax    bench/bpd_cpu.c:5370-5433
-//   SwiGLU, residual add, argmax (lowest index)    bench/bpd_cpu.c:5504-5507, 5466, 4512-4529
+//   SwiGLU, residual add                           bench/bpd_cpu.c:5504-5507, 5466
+//   argmax (lowest index), in decode_ops.cu        bench/bpd_cpu.c:4512-4529
 // Weights, caches and activations are device memory; the descriptor structs are host memory holding
 // device pointers, with the reference's field order.  Everything runs on one stream in the reference's
 // order; no kernel waits on another.  The small kernels are launched programmatically like the products: each lets the
@@ -13,6 +14,7 @@
 // launch ahead of it before it touches memory, so activations and caches are read with plain loads, never through
 // the read-only path (only weights are).
 #include "bpdq_common.cuh"
+#include "launch.cuh"
 #include "../../include/bpdq.h"
 
 #include <cuda_fp16.h>
@@ -404,61 +406,6 @@ __global__ void __launch_bounds__(256) k_add_f32(const float* a, const float* b,
         dst[i] = __fadd_rn(a[i], b[i]);
 }
 
-// One CTA per row; the largest value wins, the lowest index among equals (v > best in index order).
-__global__ void __launch_bounds__(256) k_argmax_rows(const float* x, long long* out, int n)
-{
-    pdl_launch_dependents();
-    pdl_wait();
-    __shared__ float s_v[256];
-    __shared__ int s_i[256];
-    const float* row = x + (size_t)blockIdx.x * n;
-    float best = row[0];
-    int bi = 0;
-    for (int k = threadIdx.x; k < n; k += 256) {
-        const float v = row[k];
-        if (v > best || (v == best && k < bi)) { best = v; bi = k; }
-    }
-    s_v[threadIdx.x] = best;
-    s_i[threadIdx.x] = bi;
-    __syncthreads();
-    for (int o = 128; o > 0; o >>= 1) {
-        if (threadIdx.x < o) {
-            const float v = s_v[threadIdx.x + o];
-            const int i = s_i[threadIdx.x + o];
-            if (v > s_v[threadIdx.x] || (v == s_v[threadIdx.x] && i < s_i[threadIdx.x])) {
-                s_v[threadIdx.x] = v;
-                s_i[threadIdx.x] = i;
-            }
-        }
-        __syncthreads();
-    }
-    if (threadIdx.x == 0) out[blockIdx.x] = s_i[0];
-}
-
-// A launch that may be scheduled while the launch ahead of it on the stream still runs (every kernel here waits for that
-// launch before it touches memory).
-template <typename... KArgs, typename... Args>
-static int launch_ordered(void (*kern)(KArgs...), int grid, int block, size_t smem, cudaStream_t s, Args... args)
-{
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((unsigned)grid);
-    cfg.blockDim = dim3((unsigned)block);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = s;
-    cudaLaunchAttribute at[1];
-    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = at;
-    cfg.numAttrs = tuning().pdl ? 1 : 0;
-    return check_cuda(cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...));
-}
-
-static int grid_1d(long n)
-{
-    long want = (n + 255) / 256, cap = (long)sm_count() * 8;
-    return (int)(want < 1 ? 1 : (want < cap ? want : cap));
-}
-
 static int launch_attn(const float* q, const void* kc, const void* vc, float* dst, int n_q, int n_kv, int H, int HKV, int D,
                        float scale, int kv_offset, int f16, cudaStream_t s)
 {
@@ -666,15 +613,6 @@ int bpd_swiglu_fuse_cuda(const float* gate, const float* up, float* dst, int n, 
     int rc = check_cuda(cudaGetLastError());
     return rc ? latch(rc) : 0;
 }
-int bpd_argmax_dim_cuda(const float* x, long long* out, int outer, int dim_size, int inner, void* stream)
-{
-    if (outer < 0 || dim_size < 1 || inner != 1 || (outer > 0 && (!x || !out))) return latch(BPDQ_ERR_ARG);
-    if (outer == 0) return 0;
-    launch_ordered(k_argmax_rows, outer, 256, 0, (cudaStream_t)stream, x, out, dim_size);
-    int rc = check_cuda(cudaGetLastError());
-    return rc ? latch(rc) : 0;
-}
-
 int bpd_llama_block_cuda(float* x, const bpd_llama_layer_weights* lw, const bpd_llama_config* cfg, const int32_t* pos_ids,
                          int n_tokens, int kv_pos, void* k_cache, void* v_cache, float* scratch1, float* scratch2,
                          float* scratch3, const float* rope_freqs, void* stream)
@@ -726,7 +664,7 @@ static int llama_forward(const int32_t* token_ids, int n_tokens, const bpd_llama
     if (cfg->n_layers == 0) launch_ordered(k_rmsnorm_llama, n_tokens, 256, 0, s, x, weights->output_norm_w, s1, E, cfg->rms_eps);
     if ((rc = product(weights->output_w, tiles ? tiles->output_w : nullptr, s1, logits_out, n_tokens, cfg->vocab_size, E, s, ws)))
         return rc;
-    if (token_out) launch_ordered(k_argmax_rows, n_tokens, 256, 0, s, logits_out, token_out, cfg->vocab_size);
+    if (token_out && (rc = bpd_argmax_dim_cuda(logits_out, token_out, n_tokens, cfg->vocab_size, 1, s))) return rc;
     rc = check_cuda(cudaGetLastError());
     return rc ? latch(rc) : 0;
 }

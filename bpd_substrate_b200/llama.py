@@ -3,14 +3,16 @@
 call sequence of its C-loop wrapper (inference/llamatov_c_inference.py:62-78): prefill once, then one
 token per step against the f16 KV cache.
 
-``SyntheticLlama`` makes a random model of a given shape on the host (Q8_0 matrices, norm weights);
-``DeviceLlama`` uploads one and runs ``bpd_llama_forward_cuda`` on it.  There is no CPU path here.
+``SyntheticLlama`` makes a random model of a given shape on the host (Q8_0 matrices, norm weights), ``GgufLlama``
+reads one from a GGUF file; ``DeviceLlama`` uploads one and runs ``bpd_llama_forward_cuda`` on it: with its own cache
+(``forward``) or on a sequence of the engine (``step``).  There is no CPU path here.
 """
 import ctypes as C
 
 import numpy as np
 
 from . import capi, synth
+from .sequences import SequenceSlots, StatePart, lay_out
 
 LAYER_FIELDS = ("attn_norm_w", "w_q", "w_k", "w_v", "w_o", "ffn_norm_w", "w_gate", "w_up", "w_down")
 
@@ -70,8 +72,45 @@ class SyntheticLlama:
         return w, [layers]
 
 
+class GgufLlama(SyntheticLlama):
+    """A Q8_0 Llama from a GGUF file (llama.cpp's tensor names)."""
+
+    GGUF_NAMES = dict(attn_norm_w="attn_norm", w_q="attn_q", w_k="attn_k", w_v="attn_v", w_o="attn_output", ffn_norm_w="ffn_norm",
+                      w_gate="ffn_gate", w_up="ffn_up", w_down="ffn_down")
+
+    def __init__(self, path, max_seq_len=4096):
+        from .gguf_load import TYPE_F32, TYPE_Q8_0, GgufFile
+        g = GgufFile(path)
+        meta = g.metadata
+        if meta.get("general.architecture") != "llama":
+            raise ValueError(f"{path}: architecture {meta.get('general.architecture')!r} is not llama")
+
+        def get(name, kind):
+            if name not in g.tensors:
+                raise ValueError(f"{path}: no tensor {name}")
+            if g.tensors[name].type != kind:
+                raise ValueError(f"{path}: tensor {name} has ggml type {g.tensors[name].type}, not {kind}")
+            raw = np.array(g.raw(name))
+            return raw.view(np.float32) if kind == TYPE_F32 else raw
+
+        heads = meta["llama.attention.head_count"]
+        embd = meta["llama.embedding_length"]
+        self.cfg = make_config(meta["llama.block_count"], heads, meta.get("llama.attention.head_count_kv", heads), embd // heads,
+                               meta["llama.feed_forward_length"], g.tensors["token_embd.weight"].rows, max_seq_len,
+                               meta.get("llama.attention.layer_norm_rms_epsilon", 1e-5), meta.get("llama.rope.freq_base", 10000.0),
+                               meta.get("llama.rope.dimension_count"))
+        self.token_embd = get("token_embd.weight", TYPE_Q8_0)
+        self.layers = [{f: get(f"blk.{i}.{n}.weight", TYPE_F32 if f.endswith("norm_w") else TYPE_Q8_0) for f, n in self.GGUF_NAMES.items()}
+                       for i in range(self.cfg.n_layers)]
+        self.output_norm_w = get("output_norm.weight", TYPE_F32)
+        self.output_w = get("output.weight", TYPE_Q8_0) if "output.weight" in g.tensors else self.token_embd
+        self.rope_freqs = get("rope_freqs.weight", TYPE_F32) if "rope_freqs.weight" in g.tensors else None
+        g.close()
+
+
 class DeviceLlama:
-    """A SyntheticLlama resident on the device, with its KV caches."""
+    """A SyntheticLlama or GgufLlama resident on the device.  `forward` and `read_cache` use a KV cache of its own, made at
+    the first use; `step` runs a sequence of SequenceSlots."""
 
     def __init__(self, model, lib=None):
         self.lib = lib = lib or capi.load()
@@ -84,9 +123,10 @@ class DeviceLlama:
         self.weights = capi.LlamaWeights(self._up(model.token_embd), self.layers, self._up(model.output_norm_w),
                                          self._up(model.output_w),
                                          self._up(model.rope_freqs) if model.rope_freqs is not None else None)
-        k, v = model.kv_cache()
-        self.kv_bytes = k.nbytes
-        self.d_k, self.d_v = self._up(k), self._up(v)
+        self.vocab, self.capacity = self.cfg.vocab_size, self.cfg.max_seq_len
+        self.kv_bytes = model.kv_cache()[0].nbytes
+        self._offsets = lay_out(self.state_parts(), self.capacity).offsets
+        self._slots = self._own = None
         self.stream = lib.bpdq_stream_create()
         capi.check(lib.bpdq_last_status(), "DeviceLlama setup")
 
@@ -117,12 +157,41 @@ class DeviceLlama:
         self.tiles = capi.LlamaWeights(None, self.tile_layers, None, tile(self.weights.output_w, c.vocab_size, E), None)
         capi.check(lib.bpdq_stream_sync(self.stream))
 
+    def state_parts(self):
+        """K and V of every layer, [n_layers][max_seq_len][row]; zero where nothing has been written."""
+        return [StatePart(n, self.kv_bytes // self.capacity, rows=True) for n in ("k", "v")]
+
+    def own_sequence(self):
+        if self._own is None:
+            self._slots = SequenceSlots(self.lib, self.state_parts(), self.capacity, 1, self.stream)
+            self._own = self._slots.acquire()
+        return self._own
+
+    @property
+    def d_k(self):
+        return self.own_sequence().base + self._offsets["k"]
+
+    @property
+    def d_v(self):
+        return self.own_sequence().base + self._offsets["v"]
+
+    def step(self, seq, tokens, want=(), logits=True):
+        """Runs the next tokens of `seq`; returns (logits [len(want), vocab] or None, greedy token ids [len(want)])."""
+        pos = np.arange(seq.length, seq.length + len(tokens), dtype=np.int32)
+        out, picked = self._run(tokens, pos, seq.length, seq.base + self._offsets["k"], seq.base + self._offsets["v"])
+        seq.length += len(tokens)
+        want = list(want)
+        return (out[want] if logits else None), picked[want]
+
     def reset_cache(self):
         capi.check(self.lib.bpdq_memset_async(self.d_k, 0, self.kv_bytes, self.stream))
         capi.check(self.lib.bpdq_memset_async(self.d_v, 0, self.kv_bytes, self.stream))
 
     def forward(self, token_ids, pos_ids, kv_pos):
         """Runs the tokens through all layers; returns (logits [n, vocab], argmax tokens [n])."""
+        return self._run(token_ids, pos_ids, kv_pos, self.d_k, self.d_v)
+
+    def _run(self, token_ids, pos_ids, kv_pos, d_k, d_v):
         lib = self.lib
         token_ids = np.ascontiguousarray(token_ids, np.int32)
         pos_ids = np.ascontiguousarray(pos_ids, np.int32)
@@ -134,7 +203,7 @@ class DeviceLlama:
             lib.bpdq_h2d(d_pos, pos_ids.ctypes.data, 4 * n)
             tiles = C.byref(self.tiles) if getattr(self, "tiles", None) is not None else None
             capi.check(lib.bpd_llama_forward_tiles_cuda(d_tok, n, C.byref(self.weights), tiles, C.byref(self.cfg), d_pos, kv_pos,
-                                                        self.d_k, self.d_v, d_logits, d_out, self.stream),
+                                                        d_k, d_v, d_logits, d_out, self.stream),
                        "bpd_llama_forward_tiles_cuda")
             capi.check(lib.bpdq_stream_sync(self.stream))
             logits = np.empty((n, self.cfg.vocab_size), np.float32)
@@ -159,4 +228,6 @@ class DeviceLlama:
         for p in self._allocs:
             self.lib.bpdq_free(p)
         self._allocs = []
+        if self._slots is not None:
+            self._slots.close()
         self.lib.bpdq_stream_destroy(self.stream)

@@ -443,6 +443,78 @@ int bpd_llama_forward_ws_cuda(const int32_t* token_ids, int n_tokens, const bpd_
                               void* k_cache, void* v_cache, float* logits_out, long long* token_out, void* workspace,
                               size_t workspace_bytes, void* stream);
 
+/* ---- hybrid decoder: layers of retention, state-space duality (Mamba-2) or latent attention on bf16 weights ----
+ * Weights are bf16 [out][in]; activations bf16 or fp32 (act_bf16); residual stream, norms, scores, softmax, decays and
+ * recurrent states are fp32.  Inner sizes are padded to multiples of 16 with zero weights (the *_pad fields).
+ *
+ * Single mechanisms (device pointers; act_bf16 chooses the type of the void* activations): */
+/* out[t][n] = sum_k W[n][k] x[t][k], fp32 results; K a multiple of 16 */
+int bpd_linear_bf16_cuda(const uint16_t* W, const void* x, float* out, int n_tokens, int N, int K, int act_bf16, void* stream);
+/* Per head h and token t: S = decay S + (dt k) v^T, o = S^T q + d_skip v, from and to state [heads][key_pad][value_pad].
+ * decay[h] (and its logarithm), or exp(neg_exp_a[h] dt) with dt [tokens][heads]; q and k shared by heads / groups heads */
+int bpd_decayed_scan_cuda(const void* q, int ld_q, const void* k, int ld_k, const void* v, int ld_v, const float* decay, const float* log_decay,
+                          const float* dt, const float* neg_exp_a, const float* d_skip, float* state, void* o, int ld_o, int n_tokens, int heads,
+                          int groups, int key_pad, int value_pad, int act_bf16, void* stream);
+/* pairs (i, i + rot_dims / 2) of q and k turn by (pos + t) rot_freq[i], in place; then k *= k_scale */
+int bpd_rotate_half_qk_cuda(void* q, void* k, int ld, int n_tokens, int heads, int dim_pad, int rot_dims, const float* rot_freq, float k_scale,
+                            const int32_t* pos, int act_bf16, void* stream);
+/* out = silu(b + sum_j w[j] in[t - taps + 1 + j]) per channel; tail [taps - 1][channels]: the inputs before token 0,
+ * oldest first, moved on to the last token */
+int bpd_causal_conv_silu_cuda(const void* in, int ld_in, void* out, int n_tokens, int channels, int taps, const float* w, const float* b, float* tail,
+                              int act_bf16, void* stream);
+/* over `parts` equal parts: gate_first ? rms_norm(o silu(g)) w : rms_norm(o) silu(g) */
+int bpd_gated_norm_cuda(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int n_tokens, int heads, int value_dim,
+                        int value_pad, int parts, int gate_first, float eps, int act_bf16, void* stream);
+typedef struct {
+    int heads, dim_pad, value_pad, rank, rank_pad, rot_dims, rot_pad, q_rank, q_rank_pad;
+    float scale, eps;
+    const float* rot_freq;
+} bpdq_latent_shape;
+/* u rows [query latent | latent | key part]: normed query latent to cq, normed latent and rotated (interleaved pairs)
+ * key part to cache row *pos + t ([rank_pad | rot_pad]); cache NULL: queries only */
+int bpd_latent_prepare_cuda(const bpdq_latent_shape* shape, const void* u, int ld_u, const float* q_norm, const float* kv_norm, void* cq, void* cache,
+                            const int32_t* pos, int n_tokens, int act_bf16, void* stream);
+/* q [tokens][heads][dim_pad | rot_pad] (rotated here) against cache rows 0 .. *pos + t; context = *pos + n_tokens.
+ * w_ukv: keys [heads * dim_pad][rank_pad], then values [heads * value_pad][rank_pad]; o [tokens][heads][value_pad] */
+int bpd_latent_attention_cuda(const bpdq_latent_shape* shape, void* q, const uint16_t* w_ukv, const void* cache, void* o, const int32_t* pos,
+                              int n_tokens, int context, int act_bf16, void* stream);
+
+/* The whole model.  Descriptors are host memory holding device pointers. */
+typedef struct {
+    const float *w, *b;      /* [width_pad] */
+    float alpha;
+} bpdq_dyn_tanh;             /* tanh(alpha x) * w + b */
+enum { BPDQ_MIX_RETENTION = 0, BPDQ_MIX_MAMBA2 = 1, BPDQ_MIX_LATENT = 2 };
+typedef struct {
+    int mixer, heads, groups;
+    int key_dim, key_pad, value_dim, value_pad;       /* key: dim, state or unrotated dim */
+    int rot_dims, rot_pad, conv, norm_groups, q_rank, q_rank_pad, kv_rank, kv_rank_pad, kv_from, ff_pad;   /* kv_from -1: own latents; ff_pad 0: none */
+    float scale;                                      /* retention: of k; latent attention: of the scores */
+    const float *rot_freq, *decay, *log_decay;
+    const float *conv_w, *conv_b, *dt_bias, *neg_exp_a, *d_skip, *norm_w;    /* conv_w [taps][channels] */
+    const float *q_norm_w, *kv_norm_w;
+    const uint16_t *w_in, *w_uq, *w_ukv, *w_o, *w_gate_up, *w_down;           /* gate and up rows alternate */
+    bpdq_dyn_tanh norm1, norm1b, norm2, norm2b;
+    size_t state_offset, tail_offset, cache_offset;   /* bytes into a sequence's state */
+} bpdq_hybrid_layer;
+typedef struct {
+    int n_layers, width, width_pad, vocab, act_bf16;
+    float eps;
+    const uint16_t* embed;                            /* [vocab][width_pad], also the output head */
+    bpdq_dyn_tanh final_norm;
+} bpdq_hybrid_config;
+void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers);
+void bpdq_hybrid_destroy(void* plan);
+/* Runs n_tokens tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
+ * memory.  Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
+ * the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
+ * one-token steps as a CUDA graph per state address. */
+int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int pos, void* state, const int32_t* want, int n_want,
+                        float* residuals, int use_graph, void* stream);
+float* bpdq_hybrid_logits(void* plan);                /* device [n_want][vocab] */
+void* bpdq_hybrid_picked(void* plan);                 /* device int64 [n_want] */
+size_t bpdq_hybrid_scratch_bytes(void* plan);
+
 /* ---- row-sharded products on several GPUs without a collective.
  * The reference's decode loop runs on one GPU; with the rows of every matrix sharded over ranks (one
  * process per GPU) each rank needs the other ranks' output slices.  Instead of an all-gather after the
