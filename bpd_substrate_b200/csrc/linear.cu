@@ -99,6 +99,7 @@ __global__ void __launch_bounds__(256) k_linear_tile(Linear l, int T)
         sw[kq][row] = a.x; sw[kq + 1][row] = a.y; sw[kq + 2][row] = a.z; sw[kq + 3][row] = a.w;
         sx[kq][row] = b.x; sx[kq + 1][row] = b.y; sx[kq + 2][row] = b.z; sx[kq + 3][row] = b.w;
         __syncthreads();
+        float part[4][4] = {};      // a block's sum on its own: long sums then lose less
 #pragma unroll
         for (int k = 0; k < 16; k++) {
             const float4 wv = *reinterpret_cast<const float4*>(&sw[k][4 * tr]);
@@ -107,8 +108,12 @@ __global__ void __launch_bounds__(256) k_linear_tile(Linear l, int T)
 #pragma unroll
             for (int j = 0; j < 4; j++)
 #pragma unroll
-                for (int i = 0; i < 4; i++) acc[j][i] = fmaf(wr[i], xr[j], acc[j][i]);
+                for (int i = 0; i < 4; i++) part[j][i] = fmaf(wr[i], xr[j], part[j][i]);
         }
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) acc[j][i] += part[j][i];
         __syncthreads();
     }
 #pragma unroll

@@ -16,7 +16,7 @@ def bf16_to_f32(bits):
 
 def f32_to_bf16(x):
     """Round to nearest even; finite values."""
-    u = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    u = np.array(x, np.float32, order="C").view(np.uint32)
     return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
