@@ -142,6 +142,8 @@ def _blocks(n_blocks, size, size_pad):
 
 def _spread(a, axis, places, total):
     """Entries of `a` along `axis` moved to `places` of an axis of `total`, zeros elsewhere."""
+    if a.shape[axis] == total:         # nothing to pad: the places are 0, 1, ...
+        return a
     shape = list(a.shape)
     shape[axis] = total
     out = np.zeros(shape, a.dtype)
@@ -268,7 +270,17 @@ def synthetic_tensors(spec, seed=0):
     """Random weights of the right shapes (bf16 bits): products keep activations O(1)."""
     rng = np.random.default_rng(seed)
     from .safetensors_load import f32_to_bf16
-    out = {}
+    out, pool = {}, rng.standard_normal(1 << 20, dtype=np.float32)
+    pools = {}
+
+    def matrix(shape):
+        """Large matrices repeat a pool of a million numbers (every row at another place of it)."""
+        if shape[0] * shape[1] <= pool.size:
+            return f32_to_bf16(rng.standard_normal(shape, dtype=np.float32) / np.float32(np.sqrt(shape[1])))
+        bits = pools.setdefault(shape[1], f32_to_bf16(pool / np.float32(np.sqrt(shape[1]))))
+        start = int(rng.integers(0, pool.size))
+        return np.resize(np.roll(bits, start)[:pool.size - 7], shape)
+
     for name, shape in spec.tensor_shapes().items():
         leaf = name.rsplit(".", 1)[-1]
         if name == "embed":
@@ -286,7 +298,8 @@ def synthetic_tensors(spec, seed=0):
         elif leaf == "conv":
             v = (0.5 * rng.standard_normal(shape)).astype(np.float32)
         else:
-            v = rng.standard_normal(shape, dtype=np.float32) / np.float32(np.sqrt(shape[1]))
+            out[name] = matrix(shape)
+            continue
         out[name] = f32_to_bf16(np.asarray(v, np.float32))
     return out
 

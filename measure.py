@@ -5,6 +5,9 @@
                                                     # Q8_0 Llama forward, 8B-shaped layers: ms per decoded token
     python measure.py --llama-prefill [LAYERS] [TOKENS]
                                                     # the same layers, a prefill: rows against re-tiled weights
+    python measure.py --hybrid-once prefill|decode [WIDTH] [TOKENS] [CONTEXT]
+                                                    # a few steps of the hybrid decoder (decode: launch by launch): a
+                                                    # small case for a profiler
     python measure.py --q8-tiles [N K]
                                                     # Q8_0 many-token product on re-tiled weights (tcgen05)
                                                     # beside the row-layout kernel, 1..512 tokens
@@ -244,6 +247,171 @@ def llama_decode(lib, n_layers=4, steps=32):
     return 0 if status == 0 else 1
 
 
+# ---- hybrid decoder beside the Q8_0 Llama at equal width, depth and feed-forward
+
+def hybrid_config(width, n_layers=4, vocab=32000):
+    """Layers as a real model of that width might have them, every one with a feed-forward of 3.5 widths: retention,
+    state space, latent attention, latent attention on the third layer's latents, and so on."""
+    H = width // 128
+    ff = width * 7 // 2
+    latent = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 3 * width // 8, "scale": 192 ** -0.5,
+              "rot": {"dims": 64, "base": 500000.0}}
+    kinds = [("retention", {"heads": width // 256, "dim": 256, "vdim": 256, "rot": {"dims": 256, "base": 10000.0},
+                            "decay": [1.0 - 2.0 ** (-5 - i * 7.0 / max(1, width // 256 - 1)) for i in range(width // 256)]}),
+             ("mamba2", {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}),
+             ("latent_attention", latent), ("latent_attention", dict(latent, kv_from=2))]
+    layers = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": {"kind": "dense", "ff": ff}} for i in range(n_layers)]
+    for i, la in enumerate(layers):
+        if "kv_from" in la["mixer"]:
+            la["mixer"]["kv_from"] = i - 1
+    return {"architecture": "Gurusun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def hybrid_device(lib, width, capacity, n_layers=4, dtype="bfloat16", use_graph=True):
+    from bpd_substrate_b200 import hybrid
+    spec = hybrid.HybridSpec(hybrid_config(width, n_layers))
+    return hybrid.DeviceHybrid(spec, hybrid.ArrayTensors(hybrid.synthetic_tensors(spec, 1)), dtype=dtype, capacity=capacity, lib=lib,
+                               use_graph=use_graph)
+
+
+def hybrid_flops(spec, tokens):
+    """Multiply-adds of the products of a prompt from the start, times two (attention and recurrences included)."""
+    W, f = spec.width, 0
+    for la in spec.layers:
+        m, H = la["mixer"], la["mixer"]["heads"]
+        if la["type"] == "retention":
+            f += 2 * H * (m["dim"] + m["vdim"]) * W + H * m["vdim"] * W + 2 * H * m["dim"] * m["vdim"]
+        elif la["type"] == "mamba2":
+            f += (2 * H * m["vdim"] + 2 * m["groups"] * m["state"] + H) * W + H * m["vdim"] * W + 2 * H * m["state"] * m["vdim"]
+        else:
+            f += m["q_rank"] * (W + H * (m["dim"] + m["rot_dim"])) + H * m["vdim"] * W + H * (m["dim"] + m["vdim"]) * m["kv_rank"]
+            f += 0 if m.get("kv_from") is not None else (m["kv_rank"] + m["rot_dim"]) * W
+            f += H * (m["dim"] + m["rot_dim"] + m["vdim"]) * (tokens + 1) // 2
+        f += 3 * la["mlp"]["ff"] * W if la["mlp"] else 0
+    return 2 * f * tokens
+
+
+def hybrid_bytes_per_token(model, context):
+    """What one decoded token must read and write: weights, states (both ways), cache rows of every attention layer."""
+    spec, n = model.spec, model.weight_bytes
+    rows = {p.name: p.nbytes for p in model.parts}
+    for i, la in enumerate(spec.layers):
+        if la["type"] == "latent_attention":
+            j = la["mixer"].get("kv_from")
+            n += context * rows[f"l{i if j is None else j}.cache"]
+        else:
+            n += 2 * rows[f"l{i}.state"]
+    return n
+
+
+def hybrid_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, emit=print):
+    """Prefill and decode of the hybrid decoder and of the Llama of equal width: one JSON object per number."""
+    import ctypes as C
+    import time
+
+    from bpd_substrate_b200 import llama
+    from bpd_substrate_b200.engine import Engine
+    peak, n_layers = _peak(), 4
+    capacity = max(max(prompt_tokens), context + 2 * (steps + warmup) + 80)
+    rng = np.random.default_rng(0)
+    toks = rng.integers(0, 32000, capacity).astype(np.int32)
+    e0, e1 = lib.bpdq_event_create(), lib.bpdq_event_create()
+
+    def timed(stream, fn, n, warm):
+        for _ in range(warm):
+            fn()
+        lib.bpdq_stream_sync(stream)
+        lib.bpdq_event_record(e0, stream)
+        for _ in range(n):
+            fn()
+        lib.bpdq_event_record(e1, stream)
+        return lib.bpdq_event_elapsed_ms(e0, e1) / n
+
+    def line(**kw):
+        emit(json.dumps(dict(kw, width=width, layers=n_layers, status=lib.bpdq_last_status())), flush=True)
+
+    m = hybrid_device(lib, width, capacity, n_layers)
+    e = Engine(m, 1, portion=max(prompt_tokens))
+    for T in prompt_tokens:
+        seq = e.slots.acquire()
+
+        def prompt():
+            seq.length = 0
+            m.launch(seq, toks[:T], [T - 1])
+        ms = timed(m.stream, prompt, max(3, steps // 4), warmup)
+        e.slots.release(seq)
+        line(model="hybrid", phase="prefill", tokens=T, ms=round(ms, 4), tokens_per_s=round(T / ms * 1e3),
+             tflops=round(hybrid_flops(m.spec, T) / ms / 1e9, 1))
+    seq = e.slots.acquire()
+    for at in range(0, context, max(prompt_tokens)):
+        m.launch(seq, toks[at:min(context, at + max(prompt_tokens))])
+    ms = timed(m.stream, lambda: m.launch(seq, toks[seq.length:seq.length + 1], [0]), steps, warmup)
+    e.slots.release(seq)
+    nbytes = hybrid_bytes_per_token(m, context)
+    line(model="hybrid", phase="decode", context=context, ms_per_token=round(ms, 4), tokens_per_s=round(1e3 / ms, 1), bytes_per_token=nbytes,
+         gbs=round(nbytes / ms / 1e6, 1), pct_of_measured_peak=round(100 * nbytes / ms / 1e6 / peak, 1))
+    t0 = time.perf_counter()
+    e.generate([toks[:64].tolist()], 65)
+    t1 = time.perf_counter()
+    line(model="hybrid", phase="engine end to end, 64 prompt + 65 new tokens", tokens_per_s=round(65 / (t1 - t0), 1))
+    e.close()
+    m.close()
+
+    H = width // 128
+    cfg = llama.make_config(n_layers=n_layers, n_heads=H, n_kv_heads=H // 4, head_dim=128, ffn_dim=width * 7 // 2, vocab_size=32000, max_seq_len=capacity)
+    model = llama.SyntheticLlama(cfg, seed=3)
+    dev = llama.DeviceLlama(model, lib)
+    dev.retile()
+    dev.own_sequence()
+    d_tok, d_pos = _dev(lib, toks), _dev(lib, np.arange(capacity, dtype=np.int32))
+    top = max(prompt_tokens)
+    d_logits, d_out = lib.bpdq_alloc(4 * top * cfg.vocab_size), lib.bpdq_alloc(8 * top)
+
+    def run(first, n):
+        capi.check(lib.bpd_llama_forward_tiles_cuda(d_tok + 4 * first, n, C.byref(dev.weights), C.byref(dev.tiles), C.byref(cfg), d_pos + 4 * first, first,
+                                                    dev.d_k, dev.d_v, d_logits, d_out, dev.stream))
+    for T in prompt_tokens:
+        ms = timed(dev.stream, lambda: run(0, T), 2, 1)
+        line(model="llama Q8_0", phase="prefill", tokens=T, ms=round(ms, 4), tokens_per_s=round(T / ms * 1e3))
+    for at in range(0, context, top):
+        run(at, min(top, context - at))
+    run(context, 1)
+    capi.check(lib.bpdq_stream_sync(dev.stream))
+    capi.check(lib.bpdq_graph_begin(dev.stream), "graph capture")
+    run(context, 1)
+    graph = lib.bpdq_graph_end(dev.stream)
+    ms = timed(dev.stream, lambda: capi.check(lib.bpdq_graph_launch(graph, dev.stream)), steps, warmup)
+    lib.bpdq_graph_destroy(graph)
+    nbytes = (sum(sum(v.nbytes for k, v in la.items() if k.startswith("w_")) for la in model.layers) + model.output_w.nbytes
+              + n_layers * 2 * context * cfg.n_kv_heads * 128 * 2)
+    line(model="llama Q8_0", phase="decode", context=context, ms_per_token=round(ms, 4), tokens_per_s=round(1e3 / ms, 1), bytes_per_token=nbytes,
+         gbs=round(nbytes / ms / 1e6, 1), pct_of_measured_peak=round(100 * nbytes / ms / 1e6 / peak, 1))
+    dev.close()
+    for p in (d_tok, d_pos, d_logits, d_out):
+        lib.bpdq_free(p)
+    return lib.bpdq_last_status()
+
+
+def hybrid_once(lib, phase, width=2048, tokens=1024, context=2048, repeats=2):
+    """`repeats` prompts, or one-token steps launched one kernel after the other: nothing else on the device."""
+    from bpd_substrate_b200.engine import Engine
+    m = hybrid_device(lib, width, max(tokens, context + repeats + 1), use_graph=False)
+    e = Engine(m, 1, portion=4096)
+    toks = np.random.default_rng(0).integers(0, 32000, max(tokens, context + repeats))
+    if phase == "prefill":
+        for i in range(repeats):
+            e.feed(i, toks[:tokens], [tokens - 1], logits=False)
+            e.end(i)
+    else:
+        e.feed(0, toks[:context], [], logits=False)
+        for i in range(repeats):
+            e.feed(0, toks[context + i:context + i + 1], [0], logits=False)
+    print(json.dumps({"hybrid_once": phase, "width": width, "status": lib.bpdq_last_status()}))
+    e.close()
+    m.close()
+    return 0
+
+
 def main():
     lib = capi.load()
     lib.bpdq_clear_status()
@@ -251,6 +419,8 @@ def main():
         return llama_decode(lib, *[int(v) for v in sys.argv[2:3]])
     if len(sys.argv) >= 2 and sys.argv[1] == "--llama-prefill":
         return llama_prefill(lib, *[int(v) for v in sys.argv[2:4]])
+    if len(sys.argv) >= 3 and sys.argv[1] == "--hybrid-once":
+        return hybrid_once(lib, sys.argv[2], *[int(v) for v in sys.argv[3:6]])
     if len(sys.argv) >= 2 and sys.argv[1] == "--q8-tiles":
         return q8_tiles(lib, *[int(v) for v in sys.argv[2:4]])
     if len(sys.argv) >= 3 and sys.argv[1] == "--q8-tiles-once":
