@@ -401,43 +401,42 @@ int decayed_scan(const DecayedScan& a, int T, bool act_bf16, cudaStream_t s)
 
 // ------------------------------------------------------------------ rotary positions, rotate-half pairs
 
+// Thread = (token, pair or unrotated entry of a head), all heads: one sine and cosine for all of them.
 template <typename A>
-__global__ void __launch_bounds__(256) k_rotate_half_qk(A* q, A* k, int ld, int heads, int dim_pad, int rot_dims,
-                                                        const float* __restrict__ freq, float k_scale, const int* pos, int T)
+__global__ void __launch_bounds__(128) k_rotate_half_qk(A* q, A* k, int ld, int heads, int dim_pad, int rot_dims,
+                                                        const float* __restrict__ freq, float k_scale, const int* pos)
 {
     pdl_launch_dependents();
     pdl_wait();
-    const int half = rot_dims / 2, rest = dim_pad - rot_dims, per = half + rest;    // `rest`: k's unrotated entries are scaled too
-    const long total = (long)T * heads * per;
-    const int base = *pos;
-    for (long u = (long)blockIdx.x * blockDim.x + threadIdx.x; u < total; u += (long)gridDim.x * blockDim.x) {
-        const int i = (int)(u % per);
-        const long th = u / per;
-        const int t = (int)(th / heads), h = (int)(th - (long)t * heads);
-        A* pq = q + (size_t)t * ld + h * dim_pad;
-        A* pk = k + (size_t)t * ld + h * dim_pad;
-        if (i < half) {
-            float sn, cs;
-            sincosf((float)(base + t) * freq[i], &sn, &cs);
+    const int half = rot_dims / 2, per = dim_pad - half, t = blockIdx.y;
+    const int i = blockIdx.x * 128 + threadIdx.x;
+    if (i >= per) return;
+    A* pq = q + (size_t)t * ld;
+    A* pk = k + (size_t)t * ld;
+    if (i < half) {
+        float sn, cs;
+        sincosf((float)(*pos + t) * freq[i], &sn, &cs);
+#pragma unroll 4
+        for (int h = 0; h < heads; h++, pq += dim_pad, pk += dim_pad) {
             const float q0 = act_load(pq + i), q1 = act_load(pq + i + half), k0 = act_load(pk + i), k1 = act_load(pk + i + half);
             pq[i] = act_from<A>(q0 * cs - q1 * sn);
             pq[i + half] = act_from<A>(q1 * cs + q0 * sn);
             pk[i] = act_from<A>((k0 * cs - k1 * sn) * k_scale);
             pk[i + half] = act_from<A>((k1 * cs + k0 * sn) * k_scale);
-        } else {
-            const int n = rot_dims + i - half;
-            pk[n] = act_from<A>(act_load(pk + n) * k_scale);
         }
+    } else {
+        const int n = half + i;         // k's unrotated entries are scaled too
+        for (int h = 0; h < heads; h++, pk += dim_pad) pk[n] = act_from<A>(act_load(pk + n) * k_scale);
     }
 }
 
 int rotate_half_qk(void* q, void* k, int ld, int heads, int dim_pad, int rot_dims, const float* rot_freq, float k_scale,
                    const int* pos, int T, bool act_bf16, cudaStream_t s)
 {
-    const int grid = grid_1d((long)T * heads * (dim_pad - rot_dims / 2));
+    const dim3 grid((dim_pad - rot_dims / 2 + 127) / 128, T);
     if (act_bf16)
-        return launch_ordered(k_rotate_half_qk<bf16>, grid, 256, 0, s, (bf16*)q, (bf16*)k, ld, heads, dim_pad, rot_dims, rot_freq, k_scale, pos, T);
-    return launch_ordered(k_rotate_half_qk<float>, grid, 256, 0, s, (float*)q, (float*)k, ld, heads, dim_pad, rot_dims, rot_freq, k_scale, pos, T);
+        return launch_ordered(k_rotate_half_qk<bf16>, grid, 128, 0, s, (bf16*)q, (bf16*)k, ld, heads, dim_pad, rot_dims, rot_freq, k_scale, pos);
+    return launch_ordered(k_rotate_half_qk<float>, grid, 128, 0, s, (float*)q, (float*)k, ld, heads, dim_pad, rot_dims, rot_freq, k_scale, pos);
 }
 
 // ------------------------------------------------------------------ causal convolution
@@ -523,7 +522,7 @@ int causal_conv(const void* in, int ld_in, void* out, int channels, int taps, co
 
 // ------------------------------------------------------------------ gate and norm
 
-// One CTA per (part, token).  Values are kept in registers up to 16 per thread, else computed again.
+// Any sizes: one CTA per (part, token).  Values are kept in registers up to 16 per thread, else computed again.
 template <typename A>
 __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const float* __restrict__ w, A* y,
                                                     int ld_y, int heads, int value_dim, int value_pad, int part, int gate_first, float eps)
@@ -597,19 +596,78 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
     }
 }
 
+// Unpadded heads, parts of whole groups of four: W warps per (part, token), four channels per lane and load, at most
+// eight loads per lane.
+template <typename A, int W>
+__global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, const A* g, int ld_g, const float* __restrict__ w, A* y, int ld_y,
+                                                        int part, int parts, int T, int gate_first, float eps)
+{
+    __shared__ float s_part[8];
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const long unit = (long)blockIdx.x * (8 / W) + warp / W;
+    const int t = (int)(unit / parts), first = (int)(unit - (long)t * parts) * part;
+    const bool live = t < T;
+    const int at = 4 * (lane + 32 * (warp % W)), step = 128 * W;
+    pdl_wait();
+    float4 v[8], z[8];
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        const int i = at + step * j;
+        const bool in = live && i < part;
+        v[j] = in ? act_load4(o + (size_t)t * ld_o + first + i) : make_float4(0, 0, 0, 0);
+        z[j] = in ? act_load4(g + (size_t)t * ld_g + first + i) : make_float4(0, 0, 0, 0);
+    }
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        z[j] = make_float4(silu_f32(z[j].x), silu_f32(z[j].y), silu_f32(z[j].z), silu_f32(z[j].w));
+        if (gate_first) v[j] = make_float4(v[j].x * z[j].x, v[j].y * z[j].y, v[j].z * z[j].z, v[j].w * z[j].w);
+        sum = fmaf(v[j].x, v[j].x, sum); sum = fmaf(v[j].y, v[j].y, sum); sum = fmaf(v[j].z, v[j].z, sum); sum = fmaf(v[j].w, v[j].w, sum);
+    }
+    sum = warp_sum(sum);
+    if (W > 1) {
+        if (lane == 0) s_part[warp] = sum;
+        __syncthreads();
+        sum = 0.0f;
+#pragma unroll
+        for (int i = 0; i < W; i++) sum += s_part[warp / W * W + i];
+    }
+    const float scale = 1.0f / sqrtf(sum / (float)part + eps);
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        const int i = at + step * j;
+        if (live && i < part) {
+            const float4 f = gate_first ? *reinterpret_cast<const float4*>(w + first + i) : z[j];
+            act_store4(y + (size_t)t * ld_y + first + i, make_float4(v[j].x * scale * f.x, v[j].y * scale * f.y, v[j].z * scale * f.z, v[j].w * scale * f.w));
+        }
+    }
+}
+
+template <typename A>
+static int launch_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const float* w, A* y, int ld_y, int heads, int value_dim, int value_pad,
+                             int parts, int gate_first, float eps, int T, cudaStream_t s)
+{
+    const int part = heads * value_dim / parts;
+    const bool vec = value_dim == value_pad && part % 4 == 0 && ld_o % 4 == 0 && ld_g % 4 == 0 && ld_y % 4 == 0;
+    const long units = (long)T * parts;
+    // a single token has few parts: spread one over the CTA's warps
+    if (vec && part <= 1024 && units > 64)
+        return launch_ordered(k_gated_norm_vec<A, 1>, (unsigned)((units + 7) / 8), 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+    if (vec && part <= 8192)
+        return launch_ordered(k_gated_norm_vec<A, 8>, (unsigned)units, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+    int threads = (part / 4 + 31) / 32 * 32;
+    threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;
+    return launch_ordered(k_gated_norm<A>, dim3(parts, T), threads, 0, s, o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, part, gate_first, eps);
+}
+
 int gated_norm(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int heads, int value_dim,
                int value_pad, int parts, int gate_first, float eps, int T, bool act_bf16, cudaStream_t s)
 {
-    const int inner = heads * value_dim;
-    if (parts < 1 || inner % parts || (gate_first && !w)) return latch(BPDQ_ERR_ARG);
-    const int part = inner / parts;
-    int threads = (part / 4 + 31) / 32 * 32;
-    threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;
+    if (parts < 1 || heads * value_dim % parts || (gate_first && !w)) return latch(BPDQ_ERR_ARG);
     if (act_bf16)
-        return launch_ordered(k_gated_norm<bf16>, dim3(parts, T), threads, 0, s, (const bf16*)o, ld_o, (const bf16*)g, ld_g, w, (bf16*)y, ld_y,
-                              heads, value_dim, value_pad, part, gate_first, eps);
-    return launch_ordered(k_gated_norm<float>, dim3(parts, T), threads, 0, s, (const float*)o, ld_o, (const float*)g, ld_g, w, (float*)y, ld_y,
-                          heads, value_dim, value_pad, part, gate_first, eps);
+        return launch_gated_norm((const bf16*)o, ld_o, (const bf16*)g, ld_g, w, (bf16*)y, ld_y, heads, value_dim, value_pad, parts, gate_first, eps, T, s);
+    return launch_gated_norm((const float*)o, ld_o, (const float*)g, ld_g, w, (float*)y, ld_y, heads, value_dim, value_pad, parts, gate_first, eps, T, s);
 }
 
 }  // namespace bpdq

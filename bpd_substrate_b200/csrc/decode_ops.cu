@@ -97,34 +97,44 @@ __global__ void __launch_bounds__(1024) k_matmul_f32(const float* __restrict__ A
 }
 
 // One CTA per row; the largest value wins, the lowest index among equals (v > best in index order).
-__global__ void __launch_bounds__(256) k_argmax_rows(const float* x, long long* out, int n)
+__global__ void __launch_bounds__(1024) k_argmax_rows(const float* x, long long* out, int n)
 {
     pdl_launch_dependents();
     pdl_wait();
-    __shared__ float s_v[256];
-    __shared__ int s_i[256];
+    __shared__ float s_v[32];
+    __shared__ int s_i[32];
     const float* row = x + (size_t)blockIdx.x * n;
     float best = row[0];
     int bi = 0;
-    for (int k = threadIdx.x; k < n; k += 256) {
-        const float v = row[k];
-        if (v > best || (v == best && k < bi)) { best = v; bi = k; }
+    auto better = [](float v, int k, float& bv, int& bk) {
+        if (v > bv || (v == bv && k < bk)) { bv = v; bk = k; }
+    };
+    for (int k0 = threadIdx.x; k0 < n; k0 += 8 * 1024) {
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) v[j] = k0 + 1024 * j < n ? row[k0 + 1024 * j] : row[0];
+#pragma unroll
+        for (int j = 0; j < 8; j++) better(v[j], k0 + 1024 * j < n ? k0 + 1024 * j : 0, best, bi);
     }
-    s_v[threadIdx.x] = best;
-    s_i[threadIdx.x] = bi;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xFFFFFFFFu, best, o);
+        const int i = __shfl_xor_sync(0xFFFFFFFFu, bi, o);
+        better(v, i, best, bi);
+    }
+    if ((threadIdx.x & 31) == 0) { s_v[threadIdx.x >> 5] = best; s_i[threadIdx.x >> 5] = bi; }
     __syncthreads();
-    for (int o = 128; o > 0; o >>= 1) {
-        if (threadIdx.x < o) {
-            const float v = s_v[threadIdx.x + o];
-            const int i = s_i[threadIdx.x + o];
-            if (v > s_v[threadIdx.x] || (v == s_v[threadIdx.x] && i < s_i[threadIdx.x])) {
-                s_v[threadIdx.x] = v;
-                s_i[threadIdx.x] = i;
-            }
+    if (threadIdx.x < 32) {
+        best = s_v[threadIdx.x];
+        bi = s_i[threadIdx.x];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v = __shfl_xor_sync(0xFFFFFFFFu, best, o);
+            const int i = __shfl_xor_sync(0xFFFFFFFFu, bi, o);
+            better(v, i, best, bi);
         }
-        __syncthreads();
+        if (threadIdx.x == 0) out[blockIdx.x] = bi;
     }
-    if (threadIdx.x == 0) out[blockIdx.x] = s_i[0];
 }
 
 static int ew_grid(long n)
@@ -187,7 +197,7 @@ int bpd_argmax_dim_cuda(const float* x, long long* out, int outer, int dim_size,
 {
     if (outer < 0 || dim_size < 1 || inner != 1 || (outer > 0 && (!x || !out))) return latch(BPDQ_ERR_ARG);
     if (outer == 0) return 0;
-    launch_ordered(k_argmax_rows, outer, 256, 0, (cudaStream_t)stream, x, out, dim_size);
+    launch_ordered(k_argmax_rows, outer, 1024, 0, (cudaStream_t)stream, x, out, dim_size);
     int rc = check_cuda(cudaGetLastError());
     return rc ? latch(rc) : 0;
 }

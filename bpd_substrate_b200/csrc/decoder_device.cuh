@@ -80,6 +80,13 @@ __device__ __forceinline__ float4 act_load4(const bf16* p)
                        __uint_as_float(u.y & 0xFFFF0000u));
 }
 
+__device__ __forceinline__ void act_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void act_store4(bf16* p, float4 v)
+{
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float dyn_tanh(const DynTanh& p, int n, float v) { return fmaf(tanhf(p.alpha * v), p.w[n], p.b[n]); }

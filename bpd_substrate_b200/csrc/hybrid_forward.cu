@@ -22,23 +22,21 @@
 
 namespace bpdq {
 
-// Thread = (token, column): the residual stream and the first sublayer's normed input.
+// grid (columns / 1024, tokens), four columns per thread: the residual stream and the first sublayer's normed input.
 template <typename A>
 __global__ void __launch_bounds__(256) k_embed_norm(const bf16* __restrict__ table, const int32_t* tokens, float* x, A* h, DynTanh norm, int width,
-                                                    int vocab, int T, int* err)
+                                                    int vocab, int* err)
 {
     pdl_launch_dependents();
     pdl_wait();
-    const long total = (long)T * width;
-    for (long u = (long)blockIdx.x * blockDim.x + threadIdx.x; u < total; u += (long)gridDim.x * blockDim.x) {
-        const int t = (int)(u / width), c = (int)(u - (long)t * width);
-        const int tok = tokens[t];
-        float v = 0.0f;
-        if (tok >= 0 && tok < vocab) v = __bfloat162float(table[(size_t)tok * width + c]);
-        else if (c == 0 && err) atomicCAS(err, 0, 21);      // no such row: nothing is read, code 21 is recorded
-        x[u] = v;
-        h[u] = act_from<A>(dyn_tanh(norm, c, v));
-    }
+    const int t = blockIdx.y, c = 4 * (blockIdx.x * 256 + threadIdx.x);
+    if (c >= width) return;
+    const int tok = tokens[t];
+    float4 v = make_float4(0, 0, 0, 0);
+    if (tok >= 0 && tok < vocab) v = act_load4(table + (size_t)tok * width + c);
+    else if (c == 0 && err) atomicCAS(err, 0, 21);      // no such row: nothing is read, code 21 is recorded
+    *reinterpret_cast<float4*>(x + (size_t)t * width + c) = v;
+    act_store4(h + (size_t)t * width + c, make_float4(dyn_tanh(norm, c, v.x), dyn_tanh(norm, c + 1, v.y), dyn_tanh(norm, c + 2, v.z), dyn_tanh(norm, c + 3, v.w)));
 }
 
 template <typename A>
@@ -282,8 +280,8 @@ struct Runner {
         const int W = p.cfg.width_pad, n = (int)p.layers.size();
         const bf16* table = reinterpret_cast<const bf16*>(p.cfg.embed);
         const DynTanh first = norm_of(n ? p.layers[0].norm1 : p.cfg.final_norm);
-        int rc = p.bf16_acts ? launch_ordered(k_embed_norm<bf16>, grid_1d((long)T * W), 256, 0, s, table, (const int32_t*)b.ids, b.x, (bf16*)b.h, first, W, p.cfg.vocab, T, device_error_flag())
-                             : launch_ordered(k_embed_norm<float>, grid_1d((long)T * W), 256, 0, s, table, (const int32_t*)b.ids, b.x, (float*)b.h, first, W, p.cfg.vocab, T, device_error_flag());
+        int rc = p.bf16_acts ? launch_ordered(k_embed_norm<bf16>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (bf16*)b.h, first, W, p.cfg.vocab, device_error_flag())
+                             : launch_ordered(k_embed_norm<float>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (float*)b.h, first, W, p.cfg.vocab, device_error_flag());
         if (rc) return rc;
         for (int i = 0; i < n; i++) {
             const bpdq_hybrid_layer& l = p.layers[i];
@@ -388,6 +386,7 @@ int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int 
     Plan* p = (Plan*)plan;
     cudaStream_t s = (cudaStream_t)stream;
     if (!p || !token_ids || n_tokens < 1 || pos < 0 || !state || n_want < 0 || (n_want && !want)) return latch(BPDQ_ERR_ARG);
+    if (n_tokens > 65535) return latch(BPDQ_ERR_RANGE);       // tokens are a grid dimension
     bool all = n_want == n_tokens;
     for (int i = 0; i < n_want; i++) {
         if (want[i] < 0 || want[i] >= n_tokens) return latch(BPDQ_ERR_RANGE);

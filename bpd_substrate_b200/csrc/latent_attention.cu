@@ -36,8 +36,10 @@ __global__ void __launch_bounds__(256) k_latent_prepare(LatentShape p, const A* 
     const A* row = u + (size_t)t * ld_u;
     const A* lat = row + p.q_rank_pad;
     float sq = 0.0f, sc = 0.0f;
+#pragma unroll 8
     for (int i = tid; i < p.q_rank; i += 256) { const float v = act_load(row + i); sq = fmaf(v, v, sq); }
     if (cache)
+#pragma unroll 4
         for (int i = tid; i < p.rank; i += 256) { const float v = act_load(lat + i); sc = fmaf(v, v, sc); }
     sq = warp_sum(sq);
     sc = warp_sum(sc);
@@ -47,6 +49,7 @@ __global__ void __launch_bounds__(256) k_latent_prepare(LatentShape p, const A* 
 #pragma unroll
     for (int i = 0; i < 8; i++) { sq += s_q[i]; sc += s_c[i]; }
     const float fq = 1.0f / sqrtf(sq / (float)p.q_rank + p.eps);
+#pragma unroll 8
     for (int i = tid; i < p.q_rank_pad; i += 256)
         cq[(size_t)t * p.q_rank_pad + i] = act_from<A>(i < p.q_rank ? act_load(row + i) * fq * q_norm[i] : 0.0f);
     if (!cache) return;
@@ -77,47 +80,65 @@ int latent_prepare(const LatentShape& p, const void* u, int ld_u, const float* q
 
 // ------------------------------------------------------------------ queries in latent space
 
-constexpr int kQueryTokens = 4;
-
-// grid (rank columns / 256, heads, tokens / 4); thread = two neighbouring latent columns, W_uk rows read coalesced.
-template <typename A>
-__global__ void __launch_bounds__(128) k_latent_queries(LatentShape p, const A* q, const bf16* __restrict__ w_uk, A* out, const int* pos_p, int T)
+// grid (rank columns / 128, heads, tokens / TT), 256 threads: sixteen lanes read 128 columns of a row of W_uk, sixteen
+// rows at a time; the first eight rounds of weights are requested before the launch ahead has finished.
+template <typename A, int TT>
+__global__ void __launch_bounds__(256) k_latent_queries(LatentShape p, const A* q, const bf16* __restrict__ w_uk, A* out, const int* pos_p, int T)
 {
-    extern __shared__ float sq[];       // [kQueryTokens][dim_pad]
+    extern __shared__ float sq[];       // [TT][dim_pad], then [16][132] partial sums
+    float* red = sq + TT * p.dim_pad;
     pdl_launch_dependents();
+    const int h = blockIdx.y, t0 = blockIdx.z * TT, tid = threadIdx.x;
+    const int n_t = T - t0 < TT ? T - t0 : TT;
+    const int c = blockIdx.x * 128 + 8 * (tid & 15), phase = tid >> 4;
+    const bool live = c < p.rank_pad;
+    const bf16* w = w_uk + (size_t)h * p.dim_pad * p.rank_pad + (live ? c : 0);
+    constexpr int kAhead = 8;
+    uint4 u[kAhead];
+    const int rounds = p.dim_pad / 16;
+#pragma unroll
+    for (int i = 0; i < kAhead; i++)
+        u[i] = (live && i < rounds) ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)(phase + 16 * i) * p.rank_pad)) : make_uint4(0, 0, 0, 0);
     pdl_wait();
-    const int h = blockIdx.y, t0 = blockIdx.z * kQueryTokens, tid = threadIdx.x;
-    const int n_t = T - t0 < kQueryTokens ? T - t0 : kQueryTokens;
     const int ldq = p.heads * p.q_head();
-    for (int i = tid; i < kQueryTokens * p.dim_pad; i += 128) {
+    for (int i = tid; i < TT * p.dim_pad; i += 256) {
         const int t = i / p.dim_pad, d = i - t * p.dim_pad;
         sq[i] = t < n_t ? act_load(q + (size_t)(t0 + t) * ldq + h * p.q_head() + d) : 0.0f;
     }
     __syncthreads();
-    const int c = blockIdx.x * 256 + 2 * tid;
-    if (c < p.rank_pad) {
-        float acc[kQueryTokens][2] = {};
-        const bf16* w = w_uk + (size_t)h * p.dim_pad * p.rank_pad + c;
-#pragma unroll 16
-        for (int d = 0; d < p.dim_pad; d++) {
-            const uint32_t u = __ldg(reinterpret_cast<const uint32_t*>(w + (size_t)d * p.rank_pad));
+    float acc[TT][8] = {};
+    auto add = [&](const uint4& v, int d) {
+        const float f[8] = {bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y), bf_lo(v.z), bf_hi(v.z), bf_lo(v.w), bf_hi(v.w)};
 #pragma unroll
-            for (int t = 0; t < kQueryTokens; t++) {
-                acc[t][0] = fmaf(bf_lo(u), sq[t * p.dim_pad + d], acc[t][0]);
-                acc[t][1] = fmaf(bf_hi(u), sq[t * p.dim_pad + d], acc[t][1]);
-            }
+        for (int t = 0; t < TT; t++) {
+            const float x = sq[t * p.dim_pad + d];
+#pragma unroll
+            for (int j = 0; j < 8; j++) acc[t][j] = fmaf(f[j], x, acc[t][j]);
         }
+    };
 #pragma unroll
-        for (int t = 0; t < kQueryTokens; t++)
-            if (t < n_t) {
-                A* dst = out + ((size_t)(t0 + t) * p.heads + h) * p.row() + c;
-                dst[0] = act_from<A>(acc[t][0]);
-                dst[1] = act_from<A>(acc[t][1]);
-            }
+    for (int i = 0; i < kAhead; i++)
+        if (i < rounds) add(u[i], phase + 16 * i);
+    for (int i = kAhead; i < rounds; i++)
+        add(live ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)(phase + 16 * i) * p.rank_pad)) : make_uint4(0, 0, 0, 0), phase + 16 * i);
+#pragma unroll
+    for (int t = 0; t < TT; t++) {
+        if (t >= n_t) break;
+        *reinterpret_cast<float4*>(red + phase * 132 + 8 * (tid & 15)) = make_float4(acc[t][0], acc[t][1], acc[t][2], acc[t][3]);
+        *reinterpret_cast<float4*>(red + phase * 132 + 8 * (tid & 15) + 4) = make_float4(acc[t][4], acc[t][5], acc[t][6], acc[t][7]);
+        __syncthreads();
+        const int col = blockIdx.x * 128 + tid;
+        if (tid < 128 && col < p.rank_pad) {
+            float v = 0.0f;
+#pragma unroll
+            for (int i = 0; i < 16; i++) v += red[i * 132 + tid];
+            out[((size_t)(t0 + t) * p.heads + h) * p.row() + col] = act_from<A>(v);
+        }
+        __syncthreads();
     }
     if (blockIdx.x == 0) {
         const int pairs = p.rot_pad / 2;
-        for (int i = tid; i < n_t * pairs; i += 128) {
+        for (int i = tid; i < n_t * pairs; i += 256) {
             const int t = i / pairs, j = i - t * pairs;
             const A* src = q + (size_t)(t0 + t) * ldq + h * p.q_head() + p.dim_pad + 2 * j;
             A* dst = out + ((size_t)(t0 + t) * p.heads + h) * p.row() + p.rank_pad + 2 * j;
@@ -135,6 +156,13 @@ __global__ void __launch_bounds__(128) k_latent_queries(LatentShape p, const A* 
     }
 }
 
+template <typename A, int TT>
+static int launch_latent_queries(const LatentShape& p, const void* q, const bf16* w_uk, void* out, const int* pos, int T, cudaStream_t s)
+{
+    return launch_ordered(k_latent_queries<A, TT>, dim3((p.rank_pad + 127) / 128, p.heads, (T + TT - 1) / TT), 256,
+                          (size_t)(TT * p.dim_pad + 16 * 132) * 4, s, p, (const A*)q, w_uk, (A*)out, pos, T);
+}
+
 // ------------------------------------------------------------------ attention over latents
 
 // Keys are dealt to `splits` CTAs in whole blocks; short contexts leave the last CTAs without any.
@@ -144,10 +172,16 @@ __device__ __forceinline__ int keys_per_split(int context, int splits)
     return (blocks + splits - 1) / splits * kKeyBlock;
 }
 
-// Partial results of (row, split): [rank_pad] unnormalised sums, then maximum (log2 units) and sum of weights.
-__device__ __forceinline__ float* partial_row(float* partial, long row, int split, int splits, int rank_pad)
+// Partial results of (row, split): maximum (log2 units) and sum of weights of all splits side by side, then [rank_pad]
+// unnormalised sums per split.
+__host__ __device__ inline size_t partial_stride(int splits, int rank_pad) { return (size_t)splits * (rank_pad + 2) + 2 * (splits & 1); }
+__device__ __forceinline__ float2* partial_stats(float* partial, long row, int splits, int rank_pad)
 {
-    return partial + ((size_t)row * splits + split) * (rank_pad + 4);
+    return reinterpret_cast<float2*>(partial + (size_t)row * partial_stride(splits, rank_pad));
+}
+__device__ __forceinline__ float* partial_sums(float* partial, long row, int split, int splits, int rank_pad)
+{
+    return partial + (size_t)row * partial_stride(splits, rank_pad) + 2 * (splits + (splits & 1)) + (size_t)split * rank_pad;
 }
 
 template <int MT, int NTC>
@@ -329,18 +363,15 @@ __global__ void __launch_bounds__(256, 1) k_latent_attn_mma(LatentShape p, const
         for (int e = 0; e < 4; e += 2) {
             const long g = r0 + 16 * m + g4 + 4 * e;
             if (g >= rows) continue;
-            float* dst = partial_row(partial, g, split, splits, p.rank_pad);
+            float* dst = partial_sums(partial, g, split, splits, p.rank_pad);
 #pragma unroll
             for (int n = 0; n < NTC; n++) {
                 const int c = col0 + 8 * NTC * warp + 8 * n + 2 * t4;
                 if (c < p.rank_pad && k_begin < k_end) *reinterpret_cast<float2*>(dst + c) = make_float2(o[m][n][e], o[m][n][e + 1]);
             }
         }
-    if (tid < M && r0 + tid < rows && blockIdx.z == 0) {
-        float* dst = partial_row(partial, r0 + tid, split, splits, p.rank_pad);
-        dst[p.rank_pad] = sMax[tid];
-        dst[p.rank_pad + 1] = sSum[tid];
-    }
+    if (tid < M && r0 + tid < rows && blockIdx.z == 0)
+        partial_stats(partial, r0 + tid, splits, p.rank_pad)[split] = make_float2(sMax[tid], sSum[tid]);
 }
 
 // Plain form: eight rows per CTA, one per warp; lane = key for the scores, lane = column for the sums.
@@ -407,72 +438,98 @@ __global__ void __launch_bounds__(256) k_latent_attn_rows(LatentShape p, const A
         }
     }
     if (g < rows) {
-        float* dst = partial_row(partial, g, split, splits, p.rank_pad);
+        float* dst = partial_sums(partial, g, split, splits, p.rank_pad);
         if (k_begin < k_end)
 #pragma unroll
             for (int i = 0; i < kRowCols; i++)
                 if (lane + 32 * i < p.rank_pad) dst[lane + 32 * i] = acc[i];
-        if (lane == 0) {
-            dst[p.rank_pad] = mx;
-            dst[p.rank_pad + 1] = sum;
-        }
+        if (lane == 0) partial_stats(partial, g, splits, p.rank_pad)[split] = make_float2(mx, sum);
     }
 }
 
-// grid (value columns / 32, heads, tokens): joins the splits (every CTA of a head again; the sums sit in L2), then W_uv.
+// grid (value columns / 32, heads, tokens): joins the splits (every CTA of a head again; the sums sit in L2), then W_uv: a
+// warp per four value columns, whose weights are requested before the launch ahead has finished.
 template <typename A>
-__global__ void __launch_bounds__(256) k_latent_values(LatentShape p, const float* partial, int splits, const bf16* __restrict__ w_uv, A* o,
+__global__ void __launch_bounds__(256) k_latent_values(LatentShape p, float* partial, int splits, const bf16* __restrict__ w_uv, A* o,
                                                        const int* pos_p, int T)
 {
-    extern __shared__ float lat[];      // [rank_pad], then [splits] weights
-    float* sw = lat + p.rank_pad;
+    extern __shared__ __align__(16) float lat[];      // [2][rank_pad], then [splits] weights
+    float* sw = lat + 2 * p.rank_pad;
     const int h = blockIdx.y, t = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const long row = (long)t * p.heads + h;
     pdl_launch_dependents();
+    const int c0 = blockIdx.x * 32 + 4 * warp;
+    const bf16* w = w_uv + ((size_t)h * p.value_pad + c0) * p.rank_pad;
+    uint4 u[4][2];                                     // the first 512 latent columns
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int k = 8 * lane + 256 * i;
+            u[j][i] = (c0 + j < p.value_pad && k < p.rank_pad) ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)j * p.rank_pad + k)) : make_uint4(0, 0, 0, 0);
+        }
     pdl_wait();
     const int context = *pos_p + T, per = keys_per_split(context, splits);
     const int used = (context + per - 1) / per;
-    const float* base = partial + (size_t)row * splits * (p.rank_pad + 4);
-    const size_t step = p.rank_pad + 4;
+    const float2* stats = partial_stats(partial, row, splits, p.rank_pad);
     if (warp == 0) {
+        // at most 148 splits: five per lane
+        float2 st[5];
         float mx = -INFINITY;
-        for (int i = lane; i < used; i += 32) mx = fmaxf(mx, base[i * step + p.rank_pad]);
+#pragma unroll
+        for (int i = 0; i < 5; i++) {
+            st[i] = lane + 32 * i < used ? stats[lane + 32 * i] : make_float2(-INFINITY, 0.0f);
+            mx = fmaxf(mx, st[i].x);
+        }
         mx = warp_max(mx);
         float sum = 0.0f;
-        for (int i = lane; i < used; i += 32) {
-            const float m = base[i * step + p.rank_pad];
-            const float w = m == -INFINITY ? 0.0f : exp2f(m - mx);
-            sw[i] = w;
-            sum = fmaf(w, base[i * step + p.rank_pad + 1], sum);
+#pragma unroll
+        for (int i = 0; i < 5; i++) {
+            st[i].x = st[i].x == -INFINITY ? 0.0f : exp2f(st[i].x - mx);
+            sum = fmaf(st[i].x, st[i].y, sum);
         }
-        sum = warp_sum(sum);
-        const float inv = 1.0f / sum;
-        for (int i = lane; i < used; i += 32) sw[i] *= inv;
+        const float inv = 1.0f / warp_sum(sum);
+#pragma unroll
+        for (int i = 0; i < 5; i++)
+            if (lane + 32 * i < used) sw[lane + 32 * i] = st[i].x * inv;
     }
     __syncthreads();
-    for (int c = tid; c < p.rank_pad; c += 256) {
-        float v = 0.0f;
+    // even and odd splits by the two halves of the CTA, four columns per thread
+    const float* sums = partial_sums(partial, row, 0, splits, p.rank_pad);
+    for (int c = 4 * (tid & 127); c < p.rank_pad; c += 512) {
+        float4 v = make_float4(0, 0, 0, 0);
 #pragma unroll 8
-        for (int i = 0; i < used; i++) {
-            const float w = sw[i];
-            v = w != 0.0f ? fmaf(w, base[i * step + c], v) : v;     // a split without keys for this row holds no sums
+        for (int i = tid >> 7; i < used; i += 2) {
+            const float f = sw[i];
+            const float4 a = *reinterpret_cast<const float4*>(sums + (size_t)i * p.rank_pad + c);
+            if (f != 0.0f) {                           // a split without keys for this row holds no sums
+                v.x = fmaf(f, a.x, v.x); v.y = fmaf(f, a.y, v.y); v.z = fmaf(f, a.z, v.z); v.w = fmaf(f, a.w, v.w);
+            }
         }
-        lat[c] = v;
+        *reinterpret_cast<float4*>(lat + (tid >> 7) * p.rank_pad + c) = v;
     }
     __syncthreads();
-    for (int j = warp; j < 32; j += 8) {
-        const int c = blockIdx.x * 32 + j;
-        if (c >= p.value_pad) break;
-        const bf16* w = w_uv + ((size_t)h * p.value_pad + c) * p.rank_pad;
-        float v = 0.0f;
-        for (int k = 8 * lane; k < p.rank_pad; k += 256) {
-            const uint4 u = __ldg(reinterpret_cast<const uint4*>(w + k));
-            const float4 a = *reinterpret_cast<const float4*>(lat + k), b = *reinterpret_cast<const float4*>(lat + k + 4);
-            v = fmaf(bf_lo(u.x), a.x, v); v = fmaf(bf_hi(u.x), a.y, v); v = fmaf(bf_lo(u.y), a.z, v); v = fmaf(bf_hi(u.y), a.w, v);
-            v = fmaf(bf_lo(u.z), b.x, v); v = fmaf(bf_hi(u.z), b.y, v); v = fmaf(bf_lo(u.w), b.z, v); v = fmaf(bf_hi(u.w), b.w, v);
-        }
-        v = warp_sum(v);
-        if (lane == 0) o[((size_t)t * p.heads + h) * p.value_pad + c] = act_from<A>(v);
+    for (int c = tid; c < p.rank_pad; c += 256) lat[c] += lat[p.rank_pad + c];
+    __syncthreads();
+    float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    auto add = [&](const uint4& q, int k, float& v) {
+        const float4 a = *reinterpret_cast<const float4*>(lat + k), b = *reinterpret_cast<const float4*>(lat + k + 4);
+        v = fmaf(bf_lo(q.x), a.x, v); v = fmaf(bf_hi(q.x), a.y, v); v = fmaf(bf_lo(q.y), a.z, v); v = fmaf(bf_hi(q.y), a.w, v);
+        v = fmaf(bf_lo(q.z), b.x, v); v = fmaf(bf_hi(q.z), b.y, v); v = fmaf(bf_lo(q.w), b.z, v); v = fmaf(bf_hi(q.w), b.w, v);
+    };
+#pragma unroll
+    for (int i = 0; i < 2; i++)
+        if (8 * lane + 256 * i < p.rank_pad)
+#pragma unroll
+            for (int j = 0; j < 4; j++) add(u[j][i], 8 * lane + 256 * i, acc[j]);
+    for (int k = 8 * lane + 512; k < p.rank_pad; k += 256)
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+            if (c0 + j < p.value_pad) add(__ldg(reinterpret_cast<const uint4*>(w + (size_t)j * p.rank_pad + k)), k, acc[j]);
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+        const float v = warp_sum(acc[j]);
+        if (lane == 0 && c0 + j < p.value_pad) o[((size_t)t * p.heads + h) * p.value_pad + c0 + j] = act_from<A>(v);
     }
 }
 
@@ -666,7 +723,7 @@ size_t latent_partial_floats(const LatentShape& p, int T, bool act_bf16)
 {
     if (latent_expands(p, T, act_bf16)) return 0;
     const int splits = latent_splits(p, T, act_bf16 && latent_mma_fits(p, T));
-    return (size_t)T * p.heads * splits * (p.rank_pad + 4);
+    return (size_t)T * p.heads * partial_stride(splits, p.rank_pad);
 }
 
 template <int MT, int NTC>
@@ -686,8 +743,7 @@ static int attend_latents(const LatentShape& p, const void* q, const bf16* w_ukv
                           const int* pos, int T, cudaStream_t s)
 {
     constexpr bool kBf16 = sizeof(A) == 2;
-    int rc = launch_ordered(k_latent_queries<A>, dim3((p.rank_pad + 255) / 256, p.heads, (T + kQueryTokens - 1) / kQueryTokens), 128,
-                            (size_t)kQueryTokens * p.dim_pad * 4, s, p, (const A*)q, w_ukv, (A*)b.q_latent, pos, T);
+    int rc = T == 1 ? launch_latent_queries<A, 1>(p, q, w_ukv, b.q_latent, pos, T, s) : launch_latent_queries<A, 4>(p, q, w_ukv, b.q_latent, pos, T, s);
     if (rc) return rc;
     const bool mma = kBf16 && latent_mma_fits(p, T);
     const int splits = latent_splits(p, T, mma);
@@ -711,8 +767,8 @@ static int attend_latents(const LatentShape& p, const void* q, const bf16* w_ukv
     }
     if (rc) return rc;
     const bf16* w_uv = w_ukv + (size_t)p.heads * p.dim_pad * p.rank_pad;
-    return launch_ordered(k_latent_values<A>, dim3((p.value_pad + 31) / 32, p.heads, T), 256, (size_t)(p.rank_pad + splits) * 4, s, p,
-                          (const float*)b.partial, splits, w_uv, (A*)o, pos, T);
+    return launch_ordered(k_latent_values<A>, dim3((p.value_pad + 31) / 32, p.heads, T), 256, (size_t)(2 * p.rank_pad + splits) * 4, s, p,
+                          b.partial, splits, w_uv, (A*)o, pos, T);
 }
 
 int latent_attention(const LatentShape& p, void* q, const bf16* w_ukv, const void* cache, void* o, const LatentBuffers& b, const int* pos,

@@ -3,8 +3,8 @@
 // of paired rows, the step sizes and the one-token convolution of a state-space layer).  The dynamic-tanh norm needs
 // no row statistics, so no norm is a launch of its own.
 //
-//   k_linear_vec   one token: a warp streams two weight rows with 16-byte loads, the first of them before the launch
-//                  ahead has finished (weights are constant); HBM bound
+//   k_linear_vec   one token: a warp streams two weight rows at a time with 16-byte loads, the first of them before the
+//                  launch ahead has finished (weights are constant); HBM bound
 //   k_linear_tc5   several tokens, bf16: tcgen05.mma kind::f16, 128 weight rows (TMEM lanes) x up to 256 tokens
 //                  (TMEM columns) per tile, persistent CTAs, operands by tiled TMA into a 128-byte-swizzled ring, two
 //                  accumulators so that a tile's epilogue runs under the next tile's products
@@ -26,12 +26,12 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
     const int units = l.K / 8, pairs = (l.N + 1) / 2;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int stride = gridDim.x * 8;
-    int p = blockIdx.x + gridDim.x * warp;
+    int p = blockIdx.x + gridDim.x * warp;      // row pairs are dealt over the CTAs first: every SM gets its share
     pdl_launch_dependents();
     uint4 w[2][kBatch];
-    auto fetch = [&](int pair, int base) {
-        const int r1 = 2 * pair + 1 < l.N ? 2 * pair + 1 : 2 * pair;
-        const uint4* a = reinterpret_cast<const uint4*>(l.W + (size_t)(2 * pair) * l.K);
+    auto fetch = [&](int base) {
+        const int r1 = 2 * p + 1 < l.N ? 2 * p + 1 : 2 * p;
+        const uint4* a = reinterpret_cast<const uint4*>(l.W + (size_t)(2 * p) * l.K);
         const uint4* b = reinterpret_cast<const uint4*>(l.W + (size_t)r1 * l.K);
 #pragma unroll
         for (int i = 0; i < kBatch; i++) {
@@ -40,16 +40,25 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
             w[1][i] = u < units ? __ldg(b + u) : make_uint4(0, 0, 0, 0);
         }
     };
-    if (p < pairs) fetch(p, 0);
+    if (p < pairs) fetch(0);
     pdl_wait();
     const A* in = reinterpret_cast<const A*>(l.in);
     for (int j = threadIdx.x; j < 2 * units; j += 256) xs[(j & 1) * units + (j >> 1)] = act_load4(in + 4 * j);
     __syncthreads();
     bool have = true;
     for (; p < pairs; p += stride) {
+        const int row = 2 * p + lane;
+        const bool residual = l.mode == kLinResidual && lane < 2 && row < l.N;
+        float xr = 0, pw = 0, pb = 0, nw = 0, nb = 0;       // what the residual epilogue of row 2 p + lane needs, ahead of its use
+        if (residual) {
+            xr = l.x[row];
+            pw = l.post.w[row];
+            pb = l.post.b[row];
+            if (l.next.w) { nw = l.next.w[row]; nb = l.next.b[row]; }
+        }
         float acc[2] = {0.0f, 0.0f};
         for (int base = 0; base < units; base += 32 * kBatch) {
-            if (!have) fetch(p, base);
+            if (!have) fetch(base);
             have = false;
 #pragma unroll
             for (int i = 0; i < kBatch; i++) {
@@ -72,10 +81,15 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
         }
         acc[0] = warp_sum(acc[0]);
         acc[1] = warp_sum(acc[1]);
+        const float v = lane ? acc[1] : acc[0];
         if (l.mode == kLinSwiglu) {
             if (lane == 0) reinterpret_cast<A*>(l.out)[p] = act_from<A>(silu_f32(acc[0]) * acc[1]);
-        } else if (lane < 2 && 2 * p + lane < l.N) {
-            linear_store<A>(l, 0, 2 * p + lane, lane ? acc[1] : acc[0]);
+        } else if (residual) {
+            const float r = xr + fmaf(tanhf(l.post.alpha * v), pw, pb);
+            l.x[row] = r;
+            if (l.next.w) reinterpret_cast<A*>(l.out)[row] = act_from<A>(fmaf(tanhf(l.next.alpha * r), nw, nb));
+        } else if (l.mode != kLinResidual && lane < 2 && row < l.N) {
+            linear_store<A>(l, 0, row, v);
         }
     }
 }
@@ -269,6 +283,9 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                 pw = post.w[n]; pb = post.b[n];
                 if (next.w) { nw = next.w[n]; nb = next.b[n]; }
             }
+            // rows of this warp that are only rounded and stored
+            const int n_end = (n - lane) + 32;
+            const bool plain_warp = !((l.N | l.ld_out) & 1) && (l.mode == kLinAct || (l.mode == kLinSsmIn && n_end <= l.dt_row && !l.conv.w));
             for (int c0 = 0; c0 < kCols; c0 += 16) {
                 int v[16];
                 tmem_ld(ta + c0, v);
@@ -298,6 +315,16 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                         const float g = (lane & 1) ? other : keep, u = (lane & 1) ? keep : other;
                         const int t = t0 + j + (lane & 1);
                         if (live && t < T) reinterpret_cast<bf16*>(l.out)[(size_t)t * l.ld_out + n / 2] = act_from<bf16>(silu_f32(g) * u);
+                    }
+                } else if (plain_warp) {
+                    // two neighbouring rows per store: the even lane finishes even tokens, the odd lane odd ones
+#pragma unroll
+                    for (int j = 0; j < 16; j += 2) {
+                        const float keep = __int_as_float((lane & 1) ? v[j + 1] : v[j]);
+                        const float other = __shfl_xor_sync(0xFFFFFFFFu, __int_as_float((lane & 1) ? v[j] : v[j + 1]), 1);
+                        const __nv_bfloat162 two = __floats2bfloat162_rn((lane & 1) ? other : keep, (lane & 1) ? keep : other);
+                        const int t = t0 + j + (lane & 1);
+                        if (live && t < T) *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf16*>(l.out) + (size_t)t * l.ld_out + (n & ~1)) = two;
                     }
                 } else if (live) {
 #pragma unroll
@@ -366,7 +393,7 @@ int linear_forward(const Linear& l, int T, bool act_bf16, cudaStream_t s)
         if (smem > 200 * 1024) return latch(BPDQ_ERR_RANGE);
         int rc = act_bf16 ? allow_smem<k_linear_vec<bf16>>(200 * 1024) : allow_smem<k_linear_vec<float>>(200 * 1024);
         if (rc) return rc;
-        const int want = ((l.N + 1) / 2 + 7) / 8, cap = 2 * sm_count();
+        const int want = (l.N + 1) / 2, cap = 2 * sm_count();
         const int grid = want < cap ? want : cap;
         return act_bf16 ? launch_ordered(k_linear_vec<bf16>, grid, 256, smem, s, l) : launch_ordered(k_linear_vec<float>, grid, 256, smem, s, l);
     }

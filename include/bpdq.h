@@ -505,7 +505,7 @@ typedef struct {
 } bpdq_hybrid_config;
 void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers);
 void bpdq_hybrid_destroy(void* plan);
-/* Runs n_tokens tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
+/* Runs n_tokens (up to 65535) tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
  * memory.  Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
  * the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
  * one-token steps as a CUDA graph per state address. */
