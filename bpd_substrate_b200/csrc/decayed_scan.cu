@@ -596,9 +596,9 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
     }
 }
 
-// Unpadded heads, parts of whole groups of four: W warps per (part, token), four channels per lane and load, at most
-// eight loads per lane.
-template <typename A, int W>
+// Unpadded heads, parts of whole groups of four: W warps per (part, token), four channels per lane and load, at most NJ
+// loads per lane.
+template <typename A, int W, int NJ>
 __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, const A* g, int ld_g, const float* __restrict__ w, A* y, int ld_y,
                                                         int part, int parts, int T, int gate_first, float eps)
 {
@@ -610,9 +610,9 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     const bool live = t < T;
     const int at = 4 * (lane + 32 * (warp % W)), step = 128 * W;
     pdl_wait();
-    float4 v[8], z[8];
+    float4 v[NJ], z[NJ];
 #pragma unroll
-    for (int j = 0; j < 8; j++) {
+    for (int j = 0; j < NJ; j++) {
         const int i = at + step * j;
         const bool in = live && i < part;
         v[j] = in ? act_load4(o + (size_t)t * ld_o + first + i) : make_float4(0, 0, 0, 0);
@@ -620,7 +620,7 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     }
     float sum = 0.0f;
 #pragma unroll
-    for (int j = 0; j < 8; j++) {
+    for (int j = 0; j < NJ; j++) {
         z[j] = make_float4(silu_f32(z[j].x), silu_f32(z[j].y), silu_f32(z[j].z), silu_f32(z[j].w));
         if (gate_first) v[j] = make_float4(v[j].x * z[j].x, v[j].y * z[j].y, v[j].z * z[j].z, v[j].w * z[j].w);
         sum = fmaf(v[j].x, v[j].x, sum); sum = fmaf(v[j].y, v[j].y, sum); sum = fmaf(v[j].z, v[j].z, sum); sum = fmaf(v[j].w, v[j].w, sum);
@@ -635,7 +635,7 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     }
     const float scale = 1.0f / sqrtf(sum / (float)part + eps);
 #pragma unroll
-    for (int j = 0; j < 8; j++) {
+    for (int j = 0; j < NJ; j++) {
         const int i = at + step * j;
         if (live && i < part) {
             const float4 f = gate_first ? *reinterpret_cast<const float4*>(w + first + i) : z[j];
@@ -651,11 +651,17 @@ static int launch_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const f
     const int part = heads * value_dim / parts;
     const bool vec = value_dim == value_pad && part % 4 == 0 && ld_o % 4 == 0 && ld_g % 4 == 0 && ld_y % 4 == 0;
     const long units = (long)T * parts;
+    const unsigned packed = (unsigned)((units + 7) / 8), single = (unsigned)units;
     // a single token has few parts: spread one over the CTA's warps
-    if (vec && part <= 1024 && units > 64)
-        return launch_ordered(k_gated_norm_vec<A, 1>, (unsigned)((units + 7) / 8), 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+    const bool few = units <= 64;
+    if (vec && !few && part <= 256)
+        return launch_ordered(k_gated_norm_vec<A, 1, 2>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+    if (vec && !few && part <= 1024)
+        return launch_ordered(k_gated_norm_vec<A, 1, 8>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+    if (vec && part <= 2048)
+        return launch_ordered(k_gated_norm_vec<A, 8, 2>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
     if (vec && part <= 8192)
-        return launch_ordered(k_gated_norm_vec<A, 8>, (unsigned)units, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+        return launch_ordered(k_gated_norm_vec<A, 8, 8>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
     int threads = (part / 4 + 31) / 32 * 32;
     threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;
     return launch_ordered(k_gated_norm<A>, dim3(parts, T), threads, 0, s, o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, part, gate_first, eps);

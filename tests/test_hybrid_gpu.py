@@ -172,7 +172,7 @@ def test_causal_conv(lib, bf16, taps):
 
 
 @pytest.mark.parametrize("bf16", ACTS)
-@pytest.mark.parametrize("heads,V,parts,first", [(40, 16, 40, 0), (40, 16, 10, 1), (3, 40, 3, 0), (1, 16, 1, 0), (6, 24, 4, 1), (4, 32, 1, 1), (2, 5000, 2, 1), (2, 2500, 2, 0)])
+@pytest.mark.parametrize("heads,V,parts,first", [(40, 16, 40, 0), (40, 16, 10, 1), (24, 320, 24, 0), (80, 32, 1, 1), (3, 40, 3, 0), (1, 16, 1, 0), (6, 24, 4, 1), (4, 32, 1, 1), (2, 5000, 2, 1), (2, 2500, 2, 0)])
 def test_gated_norm(lib, bf16, heads, V, parts, first):
     act, rng = Act(bf16), np.random.default_rng(V)
     T, Vp, eps = 3, pad16(V), 0.01
