@@ -69,6 +69,7 @@ struct ScratchBlock {
     cudaStream_t stream;
     uint8_t* ptr;
     size_t cap;
+    bool orphan;                         // its stream has been destroyed (a later stream may get the same handle)
 };
 std::mutex g_scratch_mutex;
 std::vector<ScratchBlock> g_scratch;     // live blocks
@@ -98,7 +99,7 @@ uint8_t* scratch_take(Workspace* ws, int kind, size_t bytes, cudaStream_t s, int
     std::lock_guard<std::mutex> lock(g_scratch_mutex);
     ScratchBlock* blk = nullptr;
     for (auto& b : g_scratch)
-        if (b.dev == dev && b.kind == kind && b.stream == s) { blk = &b; break; }
+        if (!b.orphan && b.dev == dev && b.kind == kind && b.stream == s) { blk = &b; break; }
     if (blk && blk->cap >= bytes) return blk->ptr;
     // a new or larger block is an allocation: not while the stream records a graph
     cudaStreamCaptureStatus cap = cudaStreamCaptureStatusNone;
@@ -107,6 +108,14 @@ uint8_t* scratch_take(Workspace* ws, int kind, size_t bytes, cudaStream_t s, int
         *status = latch(BPDQ_ERR_CAPTURE);
         return nullptr;
     }
+    // a stream's first block: one left by a destroyed stream, if it is large enough
+    if (!blk)
+        for (auto& b : g_scratch)
+            if (b.orphan && b.dev == dev && b.kind == kind && b.cap >= bytes) {
+                b.orphan = false;
+                b.stream = s;
+                return b.ptr;
+            }
     size_t want = bytes < (1u << 20) ? (1u << 20) : bytes;
     if (blk && want < 2 * blk->cap) want = 2 * blk->cap;
     void* p = nullptr;
@@ -121,9 +130,17 @@ uint8_t* scratch_take(Workspace* ws, int kind, size_t bytes, cudaStream_t s, int
         blk->ptr = (uint8_t*)p;
         blk->cap = want;
     } else {
-        g_scratch.push_back({dev, kind, s, (uint8_t*)p, want});
+        g_scratch.push_back({dev, kind, s, (uint8_t*)p, want, false});
     }
     return (uint8_t*)p;
+}
+
+// The stream's work is over and its handle may come back as another stream: its blocks wait for a new owner.
+static void scratch_orphan(cudaStream_t s)
+{
+    std::lock_guard<std::mutex> lock(g_scratch_mutex);
+    for (auto& b : g_scratch)
+        if (!b.orphan && b.stream == s) b.orphan = true;
 }
 
 static void* dev_alloc(size_t bytes)
@@ -242,7 +259,13 @@ void* bpdq_stream_create(void)
     if (check_cuda(cudaStreamCreateWithFlags(&s, cudaStreamNonBlocking)) != 0) return nullptr;
     return (void*)s;
 }
-void bpdq_stream_destroy(void* s) { if (s) check_cuda(cudaStreamDestroy((cudaStream_t)s)); }
+void bpdq_stream_destroy(void* s)
+{
+    if (!s) return;
+    check_cuda(cudaStreamSynchronize((cudaStream_t)s));      // nothing in flight uses the scratch blocks it leaves
+    scratch_orphan((cudaStream_t)s);
+    check_cuda(cudaStreamDestroy((cudaStream_t)s));
+}
 // Work queued on `stream` after this call waits for the work that `ev` was recorded behind.
 int bpdq_stream_wait_event(void* stream, void* ev)
 {
