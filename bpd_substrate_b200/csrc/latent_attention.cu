@@ -24,7 +24,70 @@ constexpr int kKeyBlock = 64;
 
 // ------------------------------------------------------------------ latents and cache rows
 
-// One CTA per token.
+// Query latents of up to 2048 and latents of up to 1024: one CTA per token, the row in registers, the norms' weights fetched
+// before the launch ahead has finished, the key part turned while the sums are joined.
+template <typename A>
+__global__ void __launch_bounds__(256) k_latent_prepare_regs(LatentShape p, const A* u, int ld_u, const float* __restrict__ q_norm,
+                                                             const float* __restrict__ kv_norm, A* cq, A* cache, const int* pos_p)
+{
+    __shared__ float2 s_sum[8];
+    pdl_launch_dependents();
+    const int t = blockIdx.x, tid = threadIdx.x;
+    float q[8], qw[8], c[4], cw[4];
+#pragma unroll
+    for (int j = 0; j < 8; j++) qw[j] = tid + 256 * j < p.q_rank ? q_norm[tid + 256 * j] : 0.0f;
+#pragma unroll
+    for (int j = 0; j < 4; j++) cw[j] = (cache && tid + 256 * j < p.rank) ? kv_norm[tid + 256 * j] : 0.0f;
+    const bool turns = cache && tid < p.rot_pad / 2 && 2 * tid < p.rot_dims;
+    const float freq = turns ? p.rot_freq[tid] : 0.0f;
+    pdl_wait();
+    const int pos = *pos_p + t;
+    const A* row = u + (size_t)t * ld_u;
+    const A* lat = row + p.q_rank_pad;
+    float a = 0.0f, b = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) q[j] = tid + 256 * j < p.q_rank ? act_load(row + tid + 256 * j) : 0.0f;
+#pragma unroll
+    for (int j = 0; j < 4; j++) c[j] = (cache && tid + 256 * j < p.rank) ? act_load(lat + tid + 256 * j) : 0.0f;
+    if (turns) {
+        a = act_load(lat + p.rank_pad + 2 * tid);
+        b = act_load(lat + p.rank_pad + 2 * tid + 1);
+    }
+    float sq = 0.0f, sc = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) sq = fmaf(q[j], q[j], sq);
+#pragma unroll
+    for (int j = 0; j < 4; j++) sc = fmaf(c[j], c[j], sc);
+    sq = warp_sum(sq);
+    sc = warp_sum(sc);
+    if ((tid & 31) == 0) s_sum[tid >> 5] = make_float2(sq, sc);
+    if (turns) {
+        float sn, cs;
+        sincosf((float)pos * freq, &sn, &cs);
+        const float x = a;
+        a = x * cs - b * sn;
+        b = b * cs + x * sn;
+    }
+    A* dst = cache ? cache + (size_t)pos * p.row() : nullptr;
+    if (cache && tid < p.rot_pad / 2) {
+        dst[p.rank_pad + 2 * tid] = act_from<A>(a);
+        dst[p.rank_pad + 2 * tid + 1] = act_from<A>(b);
+    }
+    __syncthreads();
+    sq = sc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) { sq += s_sum[i].x; sc += s_sum[i].y; }
+    const float fq = 1.0f / sqrtf(sq / (float)p.q_rank + p.eps), fc = 1.0f / sqrtf(sc / (float)p.rank + p.eps);
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+        if (tid + 256 * j < p.q_rank_pad) cq[(size_t)t * p.q_rank_pad + tid + 256 * j] = act_from<A>(q[j] * fq * qw[j]);
+    if (!cache) return;
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+        if (tid + 256 * j < p.rank_pad) dst[tid + 256 * j] = act_from<A>(c[j] * fc * cw[j]);
+}
+
+// Any sizes: one CTA per token.
 template <typename A>
 __global__ void __launch_bounds__(256) k_latent_prepare(LatentShape p, const A* u, int ld_u, const float* __restrict__ q_norm,
                                                         const float* __restrict__ kv_norm, A* cq, A* cache, const int* pos_p)
@@ -74,6 +137,10 @@ __global__ void __launch_bounds__(256) k_latent_prepare(LatentShape p, const A* 
 int latent_prepare(const LatentShape& p, const void* u, int ld_u, const float* q_norm, const float* kv_norm, void* cq, void* cache,
                    const int* pos, int T, bool act_bf16, cudaStream_t s)
 {
+    if (p.q_rank_pad <= 2048 && p.rank_pad <= 1024 && p.rot_pad <= 512) {
+        if (act_bf16) return launch_ordered(k_latent_prepare_regs<bf16>, T, 256, 0, s, p, (const bf16*)u, ld_u, q_norm, kv_norm, (bf16*)cq, (bf16*)cache, pos);
+        return launch_ordered(k_latent_prepare_regs<float>, T, 256, 0, s, p, (const float*)u, ld_u, q_norm, kv_norm, (float*)cq, (float*)cache, pos);
+    }
     if (act_bf16) return launch_ordered(k_latent_prepare<bf16>, T, 256, 0, s, p, (const bf16*)u, ld_u, q_norm, kv_norm, (bf16*)cq, (bf16*)cache, pos);
     return launch_ordered(k_latent_prepare<float>, T, 256, 0, s, p, (const float*)u, ld_u, q_norm, kv_norm, (float*)cq, (float*)cache, pos);
 }

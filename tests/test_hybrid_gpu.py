@@ -264,9 +264,10 @@ def test_latent_attention_sizes(lib, bf16, T, pos, H, D, r, V, R):
 
 
 @pytest.mark.parametrize("bf16", ACTS)
-def test_latent_prepare(lib, bf16):
+@pytest.mark.parametrize("Q,R,r", [(300, 40, 6), (2048, 1000, 64), (2100, 40, 16), (40, 1100, 2)])
+def test_latent_prepare(lib, bf16, Q, R, r):
     act, rng = Act(bf16), np.random.default_rng(8)
-    T, pos, Q, R, r = 4, 37, 300, 40, 6
+    T, pos = 4, 37
     Qp, Rp, rp = pad16(Q), pad16(R), pad16(r)
     u = act.host(rng.standard_normal((T, Q + R + r)) * 0.05)
     us = np.zeros((T, Qp + Rp + rp), np.float32)
