@@ -126,3 +126,39 @@ def test_loaded_shards_run_through_the_kernels(lib, oracle, model_file):
         assert lib.bpdq_last_status() == 0
     finally:
         g.close()
+
+
+def test_a_llama_comes_back_from_a_gguf_file(tmp_path):
+    """GgufLlama reads what was written from a SyntheticLlama: sizes, constants, every matrix and norm."""
+    from bpd_substrate_b200 import llama
+    cfg = llama.make_config(n_layers=2, n_heads=4, n_kv_heads=2, head_dim=32, ffn_dim=96, vocab_size=70, max_seq_len=48, rms_eps=1e-6,
+                            rope_base=7000.0)
+    src = llama.SyntheticLlama(cfg, seed=5)
+    path = str(tmp_path / "m.gguf")
+    w = gguf.GGUFWriter(path, "llama")
+    for key, v in (("block_count", 2), ("attention.head_count", 4), ("attention.head_count_kv", 2), ("embedding_length", 128),
+                   ("feed_forward_length", 96), ("rope.dimension_count", 32)):
+        w.add_uint32("llama." + key, v)
+    w.add_float32("llama.attention.layer_norm_rms_epsilon", 1e-6)
+    w.add_float32("llama.rope.freq_base", 7000.0)
+    q8 = gguf.GGMLQuantizationType.Q8_0
+    w.add_tensor("token_embd.weight", src.token_embd.reshape(70, -1), raw_dtype=q8)
+    for i, layer in enumerate(src.layers):
+        for field, name in llama.GgufLlama.GGUF_NAMES.items():
+            a = layer[field]
+            rows = {"w_q": 128, "w_k": 64, "w_v": 64, "w_o": 128, "w_gate": 96, "w_up": 96, "w_down": 128}.get(field)
+            w.add_tensor(f"blk.{i}.{name}.weight", a if rows is None else a.reshape(rows, -1), raw_dtype=None if rows is None else q8)
+    w.add_tensor("output_norm.weight", src.output_norm_w)
+    w.add_tensor("output.weight", src.output_w.reshape(70, -1), raw_dtype=q8)
+    w.add_tensor("rope_freqs.weight", src.rope_freqs)
+    w.write_header_to_file()
+    w.write_kv_data_to_file()
+    w.write_tensors_to_file()
+    w.close()
+    got = llama.GgufLlama(path, max_seq_len=48)
+    for f, _ in cfg._fields_:
+        assert getattr(got.cfg, f) == getattr(cfg, f), f
+    for a, b in zip(got.layers, src.layers):
+        assert all(np.array_equal(a[f].ravel(), b[f].ravel()) for f in b)
+    for f in ("token_embd", "output_norm_w", "output_w", "rope_freqs"):
+        assert np.array_equal(getattr(got, f).ravel(), getattr(src, f).ravel()), f
