@@ -9,10 +9,11 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libbpdq.so")
 SOURCES = ["runtime.cu", "dequant_q4k.cu", "gemv_q4k.cu", "gemv_batch.cu", "gemv_persistent.cu", "gemv_stream.cu", "q8_0.cu", "w4a32.cu", "decode_ops.cu", "gemm_q4k_mma.cu", "gemm_q4k_tc5.cu", "gemm_q4k_rg16.cu", "gemm_q8_0_tiles.cu", "llama_forward.cu", "peer_exchange.cu",
-           "linear.cu", "decayed_scan.cu", "latent_attention.cu", "hybrid_forward.cu"]
-# The sources one model family needs: a process that only serves that family (bin/trace_run in a fresh checkout)
+           "linear.cu", "decayed_scan.cu", "latent_attention.cu", "delta_rule.cu", "grouped_attention.cu", "residual_streams.cu", "hybrid_forward.cu"]
+# The sources some model families need: a process that only serves one of those (bin/trace_run in a fresh checkout)
 # compiles and loads these as a library of their own when the whole one has not been built.
-PARTS = {"hybrid": ["runtime.cu", "decode_ops.cu", "linear.cu", "decayed_scan.cu", "latent_attention.cu", "hybrid_forward.cu"]}
+PARTS = {"hybrid": ["runtime.cu", "decode_ops.cu", "linear.cu", "decayed_scan.cu", "latent_attention.cu", "delta_rule.cu", "grouped_attention.cu",
+                    "residual_streams.cu", "hybrid_forward.cu"]}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",

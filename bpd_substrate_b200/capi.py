@@ -176,7 +176,11 @@ SIGNATURES = {
     "bpd_gated_norm_cuda": (i32, [vp, i32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp]),
     "bpd_latent_prepare_cuda": (i32, [vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, vp]),
     "bpd_latent_attention_cuda": (i32, [vp, vp, vp, vp, vp, vp, i32, i32, i32, vp]),
+    "bpd_delta_rule_cuda": (i32, [vp, vp, vp, i32, vp, vp, f32, f32, vp, vp, vp, vp, f32, i32, i32, i32, i32, i32, i32, i32, vp]),
+    "bpd_grouped_attention_cuda": (i32, [vp, vp, i32, vp, i32, vp, vp, i32, i32, vp]),
+    "bpd_stream_step_cuda": (i32, [vp, vp, vp, i32, vp, f32, i32, i32, i32, vp, vp, i32, vp]),
     "bpdq_hybrid_create": (vp, [vp, vp]),
+    "bpdq_hybrid_portion": (i32, [vp]),
     "bpdq_hybrid_destroy": (None, [vp]),
     "bpdq_hybrid_forward": (i32, [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp]),
     "bpdq_hybrid_logits": (vp, [vp]),
@@ -256,24 +260,40 @@ class DynTanh(C.Structure):
     _fields_ = [("w", vp), ("b", vp), ("alpha", f32)]
 
 
-MIX_RETENTION, MIX_MAMBA2, MIX_LATENT = 0, 1, 2
+class GroupedShape(C.Structure):
+    """bpdq_grouped_shape."""
+    _fields_ = [(n, i32) for n in ("heads", "groups", "dim", "dim_pad", "value_pad", "chunk", "rows", "sink")] + [(n, f32) for n in ("scale", "cap", "eps")]
+
+
+MAX_STREAMS = 8
+
+
+class StreamMix(C.Structure):
+    """bpdq_stream_mix."""
+    _fields_ = [("mix", f32 * (MAX_STREAMS * MAX_STREAMS)), ("out", f32 * MAX_STREAMS), ("in_", f32 * MAX_STREAMS)]
+
+
+MIX_RETENTION, MIX_MAMBA2, MIX_LATENT, MIX_DELTA, MIX_GROUPED = range(5)
+FF_SWIGLU, FF_GELU = range(2)
 
 
 class HybridLayer(C.Structure):
     """bpdq_hybrid_layer."""
     _fields_ = ([(n, i32) for n in ("mixer", "heads", "groups", "key_dim", "key_pad", "value_dim", "value_pad", "rot_dims", "rot_pad",
-                                    "conv", "norm_groups", "q_rank", "q_rank_pad", "kv_rank", "kv_rank_pad", "kv_from", "ff_pad")]
-                + [("scale", f32)]
+                                    "conv", "norm_groups", "q_rank", "q_rank_pad", "kv_rank", "kv_rank_pad", "kv_from", "ff_pad",
+                                    "ff_kind", "gate_rank_pad", "chunk", "cache_rows")]
+                + [("scale", f32), ("softcap", f32)]
                 + [(n, vp) for n in ("rot_freq", "decay", "log_decay", "conv_w", "conv_b", "dt_bias", "neg_exp_a", "d_skip", "norm_w",
-                                     "q_norm_w", "kv_norm_w", "w_in", "w_uq", "w_ukv", "w_o", "w_gate_up", "w_down")]
+                                     "q_norm_w", "kv_norm_w", "w_in", "w_uq", "w_ukv", "w_o", "w_gate_up", "w_down", "w_gates")]
                 + [(n, DynTanh) for n in ("norm1", "norm1b", "norm2", "norm2b")]
+                + [(n, StreamMix) for n in ("mix1", "mix2")]
                 + [(n, sz) for n in ("state_offset", "tail_offset", "cache_offset")])
 
 
 class HybridConfig(C.Structure):
     """bpdq_hybrid_config."""
-    _fields_ = [(n, i32) for n in ("n_layers", "width", "width_pad", "vocab", "act_bf16")] + [("eps", f32), ("embed", vp),
-                                                                                              ("final_norm", DynTanh)]
+    _fields_ = ([(n, i32) for n in ("n_layers", "width", "width_pad", "vocab", "act_bf16", "streams")]
+                + [(n, f32) for n in ("eps", "embed_scale", "logit_cap")] + [("embed", vp), ("head", vp), ("final_norm", DynTanh)])
 
 
 class BpdqError(RuntimeError):

@@ -453,7 +453,7 @@ __global__ void __launch_bounds__(128) k_causal_conv(const A* in, int ld_in, A* 
     const int c = blockIdx.x * 128 + threadIdx.x;
     if (c >= channels) return;
     const int t0 = blockIdx.y * kConvTile, t1 = t0 + kConvTile < T ? t0 + kConvTile : T;
-    const float bias = b[c];
+    const float bias = b ? b[c] : 0.0f;
     auto input = [&](int t) -> float {      // t >= -(taps - 1)
         return t >= 0 ? act_load(in + (size_t)t * ld_in + c) : tail[(size_t)(t + taps - 1) * channels + c];
     };
@@ -522,10 +522,13 @@ int causal_conv(const void* in, int ld_in, void* out, int channels, int taps, co
 
 // ------------------------------------------------------------------ gate and norm
 
+// What multiplies: silu, or (after a norm with a weight) sigmoid of the gate.
+__device__ __forceinline__ float gate_value(int form, float g) { return form == kNormWeightGate ? sigmoid_f32(g) : silu_f32(g); }
+
 // Any sizes: one CTA per (part, token).  Values are kept in registers up to 16 per thread, else computed again.
 template <typename A>
 __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const float* __restrict__ w, A* y,
-                                                    int ld_y, int heads, int value_dim, int value_pad, int part, int gate_first, float eps)
+                                                    int ld_y, int heads, int value_dim, int value_pad, int part, int form, float eps)
 {
     __shared__ float s_part[8];
     pdl_launch_dependents();
@@ -559,15 +562,15 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
         }
 #pragma unroll
         for (int j = 0; j < kKeep; j++) {
-            gate[j] = silu_f32(gate[j]);
-            if (gate_first) keep[j] *= gate[j];
+            gate[j] = gate_value(form, gate[j]);
+            if (form == kGateThenNorm) keep[j] *= gate[j];
             sum = fmaf(keep[j], keep[j], sum);
         }
     } else {
         for (int i = threadIdx.x; i < part; i += n) {
             const int c = where(i);
             float v = act_load(po + c);
-            if (gate_first) v *= silu_f32(act_load(pg + c));
+            if (form == kGateThenNorm) v *= silu_f32(act_load(pg + c));
             sum = fmaf(v, v, sum);
         }
     }
@@ -584,14 +587,14 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
             const int i = threadIdx.x + j * n;
             if (i < part) {
                 const int c = where(i);
-                py[c] = act_from<A>(keep[j] * scale * (gate_first ? w[c] : gate[j]));
+                py[c] = act_from<A>(keep[j] * scale * (form != kNormThenGate ? w[c] : 1.0f) * (form != kGateThenNorm ? gate[j] : 1.0f));
             }
         }
     } else {
         for (int i = threadIdx.x; i < part; i += n) {
             const int c = where(i);
-            const float v = act_load(po + c), z = silu_f32(act_load(pg + c));
-            py[c] = act_from<A>(v * z * scale * (gate_first ? w[c] : 1.0f));
+            const float v = act_load(po + c), z = gate_value(form, act_load(pg + c));
+            py[c] = act_from<A>(v * z * scale * (form != kNormThenGate ? w[c] : 1.0f));
         }
     }
 }
@@ -600,7 +603,7 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
 // loads per lane.
 template <typename A, int W, int NJ>
 __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, const A* g, int ld_g, const float* __restrict__ w, A* y, int ld_y,
-                                                        int part, int parts, int T, int gate_first, float eps)
+                                                        int part, int parts, int T, int form, float eps)
 {
     __shared__ float s_part[8];
     pdl_launch_dependents();
@@ -621,8 +624,8 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     float sum = 0.0f;
 #pragma unroll
     for (int j = 0; j < NJ; j++) {
-        z[j] = make_float4(silu_f32(z[j].x), silu_f32(z[j].y), silu_f32(z[j].z), silu_f32(z[j].w));
-        if (gate_first) v[j] = make_float4(v[j].x * z[j].x, v[j].y * z[j].y, v[j].z * z[j].z, v[j].w * z[j].w);
+        z[j] = make_float4(gate_value(form, z[j].x), gate_value(form, z[j].y), gate_value(form, z[j].z), gate_value(form, z[j].w));
+        if (form == kGateThenNorm) v[j] = make_float4(v[j].x * z[j].x, v[j].y * z[j].y, v[j].z * z[j].z, v[j].w * z[j].w);
         sum = fmaf(v[j].x, v[j].x, sum); sum = fmaf(v[j].y, v[j].y, sum); sum = fmaf(v[j].z, v[j].z, sum); sum = fmaf(v[j].w, v[j].w, sum);
     }
     sum = warp_sum(sum);
@@ -638,7 +641,11 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     for (int j = 0; j < NJ; j++) {
         const int i = at + step * j;
         if (live && i < part) {
-            const float4 f = gate_first ? *reinterpret_cast<const float4*>(w + first + i) : z[j];
+            float4 f = z[j];
+            if (form != kNormThenGate) {
+                f = *reinterpret_cast<const float4*>(w + first + i);
+                if (form == kNormWeightGate) f = make_float4(f.x * z[j].x, f.y * z[j].y, f.z * z[j].z, f.w * z[j].w);
+            }
             act_store4(y + (size_t)t * ld_y + first + i, make_float4(v[j].x * scale * f.x, v[j].y * scale * f.y, v[j].z * scale * f.z, v[j].w * scale * f.w));
         }
     }
@@ -646,7 +653,7 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
 
 template <typename A>
 static int launch_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const float* w, A* y, int ld_y, int heads, int value_dim, int value_pad,
-                             int parts, int gate_first, float eps, int T, cudaStream_t s)
+                             int parts, int form, float eps, int T, cudaStream_t s)
 {
     const int part = heads * value_dim / parts;
     const bool vec = value_dim == value_pad && part % 4 == 0 && ld_o % 4 == 0 && ld_g % 4 == 0 && ld_y % 4 == 0;
@@ -655,25 +662,25 @@ static int launch_gated_norm(const A* o, int ld_o, const A* g, int ld_g, const f
     // a single token has few parts: spread one over the CTA's warps
     const bool few = units <= 64;
     if (vec && !few && part <= 256)
-        return launch_ordered(k_gated_norm_vec<A, 1, 2>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+        return launch_ordered(k_gated_norm_vec<A, 1, 2>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, form, eps);
     if (vec && !few && part <= 1024)
-        return launch_ordered(k_gated_norm_vec<A, 1, 8>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+        return launch_ordered(k_gated_norm_vec<A, 1, 8>, packed, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, form, eps);
     if (vec && part <= 2048)
-        return launch_ordered(k_gated_norm_vec<A, 8, 2>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+        return launch_ordered(k_gated_norm_vec<A, 8, 2>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, form, eps);
     if (vec && part <= 8192)
-        return launch_ordered(k_gated_norm_vec<A, 8, 8>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, gate_first, eps);
+        return launch_ordered(k_gated_norm_vec<A, 8, 8>, single, 256, 0, s, o, ld_o, g, ld_g, w, y, ld_y, part, parts, T, form, eps);
     int threads = (part / 4 + 31) / 32 * 32;
     threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;
-    return launch_ordered(k_gated_norm<A>, dim3(parts, T), threads, 0, s, o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, part, gate_first, eps);
+    return launch_ordered(k_gated_norm<A>, dim3(parts, T), threads, 0, s, o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, part, form, eps);
 }
 
 int gated_norm(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int heads, int value_dim,
-               int value_pad, int parts, int gate_first, float eps, int T, bool act_bf16, cudaStream_t s)
+               int value_pad, int parts, int form, float eps, int T, bool act_bf16, cudaStream_t s)
 {
-    if (parts < 1 || heads * value_dim % parts || (gate_first && !w)) return latch(BPDQ_ERR_ARG);
+    if (parts < 1 || heads * value_dim % parts || form < 0 || form > 2 || (form != kNormThenGate && !w)) return latch(BPDQ_ERR_ARG);
     if (act_bf16)
-        return launch_gated_norm((const bf16*)o, ld_o, (const bf16*)g, ld_g, w, (bf16*)y, ld_y, heads, value_dim, value_pad, parts, gate_first, eps, T, s);
-    return launch_gated_norm((const float*)o, ld_o, (const float*)g, ld_g, w, (float*)y, ld_y, heads, value_dim, value_pad, parts, gate_first, eps, T, s);
+        return launch_gated_norm((const bf16*)o, ld_o, (const bf16*)g, ld_g, w, (bf16*)y, ld_y, heads, value_dim, value_pad, parts, form, eps, T, s);
+    return launch_gated_norm((const float*)o, ld_o, (const float*)g, ld_g, w, (float*)y, ld_y, heads, value_dim, value_pad, parts, form, eps, T, s);
 }
 
 }  // namespace bpdq
@@ -716,17 +723,17 @@ int bpd_causal_conv_silu_cuda(const void* in, int ld_in, void* out, int n_tokens
 {
     if (n_tokens < 0 || channels < 1 || taps < 1) return latch(BPDQ_ERR_ARG);
     if (n_tokens == 0) return 0;
-    if (!in || !out || !w || !b || (taps > 1 && !tail)) return latch(BPDQ_ERR_ARG);
+    if (!in || !out || !w || (taps > 1 && !tail)) return latch(BPDQ_ERR_ARG);
     return causal_conv(in, ld_in, out, channels, taps, w, b, tail, n_tokens, act_bf16 != 0, (cudaStream_t)stream);
 }
 
 int bpd_gated_norm_cuda(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int n_tokens, int heads, int value_dim,
-                        int value_pad, int parts, int gate_first, float eps, int act_bf16, void* stream)
+                        int value_pad, int parts, int form, float eps, int act_bf16, void* stream)
 {
     if (n_tokens < 0 || heads < 1 || value_dim < 1 || value_pad < value_dim) return latch(BPDQ_ERR_ARG);
     if (n_tokens == 0) return 0;
     if (!o || !g || !y) return latch(BPDQ_ERR_ARG);
-    return gated_norm(o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, parts, gate_first, eps, n_tokens, act_bf16 != 0, (cudaStream_t)stream);
+    return gated_norm(o, ld_o, g, ld_g, w, y, ld_y, heads, value_dim, value_pad, parts, form, eps, n_tokens, act_bf16 != 0, (cudaStream_t)stream);
 }
 
 }  // extern "C"

@@ -31,14 +31,19 @@ int decayed_scan(const DecayedScan& a, int T, bool act_bf16, cudaStream_t s);
 int rotate_half_qk(void* q, void* k, int ld, int heads, int dim_pad, int rot_dims, const float* rot_freq, float k_scale,
                    const int* pos, int T, bool act_bf16, cudaStream_t s);
 
-// Causal depthwise convolution with bias and silu over T tokens: in [T][ld_in] -> out [T][channels]; tail
+// Causal depthwise convolution with bias (b null: none) and silu over T tokens: in [T][ld_in] -> out [T][channels]; tail
 // [taps - 1][channels] (oldest first) is the window before the first token and is moved on to the last one.
 int causal_conv(const void* in, int ld_in, void* out, int channels, int taps, const float* w, const float* b, float* tail, int T,
                 bool act_bf16, cudaStream_t s);
 
 // Gate and RMS norm over `parts` equal parts of the heads' outputs (heads of value_dim stored value_pad apart):
-//   gate_first = 0: y = (o / rms(o)) * silu(g)          gate_first = 1: u = o * silu(g), y = u / rms(u) * w
+// in one of three forms; w has an entry per stored channel.
+enum GatedNormForm {
+    kNormThenGate = 0,      // y = o / rms(o) * silu(g)
+    kGateThenNorm = 1,      // u = o * silu(g), y = u / rms(u) * w
+    kNormWeightGate = 2     // y = o / rms(o) * w * sigmoid(g)
+};
 int gated_norm(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int heads, int value_dim,
-               int value_pad, int parts, int gate_first, float eps, int T, bool act_bf16, cudaStream_t s);
+               int value_pad, int parts, int form, float eps, int T, bool act_bf16, cudaStream_t s);
 
 }  // namespace bpdq

@@ -1,6 +1,5 @@
-// Building blocks shared by the kernels of the hybrid decoder (recurrent and latent-attention layers on bf16
-// weights): activation types, the dynamic-tanh norm, the epilogues of its matrix products, bf16 tensor-core
-// fragments.
+// Building blocks shared by the kernels of the hybrid decoders (recurrent and attention layers on bf16 weights):
+// activation types, the dynamic-tanh norm, the epilogues of their matrix products, bf16 tensor-core fragments.
 //
 // Weights are bf16.  Activations are bf16 or fp32 (the template parameter A); the residual stream, norms, scores,
 // softmax, decays and recurrent states are fp32 in both cases.  Every inner size is padded to a multiple of 16 with
@@ -26,13 +25,28 @@ enum LinearMode {
     kLinF32 = 1,        // out[t][n] = v
     kLinResidual = 2,   // x[t][n] += post(v); out[t][n] = A(next(x[t][n])) when `next` is given
     kLinSwiglu = 3,     // rows come in pairs (2i: gate, 2i + 1: up); out[t][i] = A(silu(gate) * up)
-    kLinSsmIn = 4       // rows >= dt_row are step sizes: dt[t][n - dt_row] = softplus(v + dt_bias) in fp32; with
-                        // conv.w also the rows of [conv_row, dt_row) pass the causal convolution (one token only)
+    kLinMixerIn = 4,    // rows >= dt_row are step sizes in fp32: dt[t][n - dt_row] = softplus(v + dt_bias), or sigmoid(v)
+                        // without a dt_bias; with conv.w also conv.channels rows from conv_row on pass the causal
+                        // convolution (one token only)
+    kLinLogDecay = 5,   // dt[t][n] = neg_exp_a[n] softplus(v + dt_bias[n]) in fp32; with split (one token only) the rows
+                        // from there on read the input from in + in2 on: out[t][n - split] = A(v)
+    kLinGelu = 6,       // out[t][n] = A(gelu(v)), tanh form
+    kLinStreams = 7     // one token only: the residual streams of column n take v in, and their sum with the next
+                        // sublayer's weights goes to u[n]
+};
+
+// Residual streams joined by hyper-connections: x_t <- sum_s mix[s][t] x_s + out[t] y; the next sublayer reads
+// sum_t next[t] x_t.
+constexpr int kMaxStreams = 8;
+struct StreamMix {
+    int n;
+    float mix[kMaxStreams][kMaxStreams];
+    float out[kMaxStreams], next[kMaxStreams];
 };
 
 // Depthwise causal convolution of one token: tail [taps - 1][channels] holds the inputs before it, oldest first.
 struct ConvStep {
-    const float *w, *b;     // w [taps][channels]; w == null: no convolution here
+    const float *w, *b;     // w [taps][channels]; w == null: no convolution here; b == null: no bias
     float* tail;
     void* out;              // [channels], activation type
     int taps, channels;
@@ -49,10 +63,17 @@ struct Linear {
     int ld_x;
     DynTanh post, next;
     int conv_row, dt_row;
-    const float* dt_bias;
+    const float *dt_bias, *neg_exp_a;
     float* dt;              // [T][ld_dt]
     int ld_dt;
     ConvStep conv;
+    int split, in2;
+    float cap;              // kLinF32: v becomes cap tanh(v / cap); 0: as it is
+    const float* norm_w;    // one token only: `in` is fp32 and passes an RMS norm with this weight over norm_n entries
+    int norm_n;
+    float norm_eps;
+    StreamMix streams;      // kLinStreams: of x [streams.n][ld_x]
+    float* u;
 };
 
 // Runs one product over T tokens (linear.cu); act_bf16: A is bf16, else fp32.
@@ -88,6 +109,12 @@ __device__ __forceinline__ void act_store4(bf16* p, float4 v)
 }
 
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f32(float z)
+{
+    // 0.5 (1 + tanh(a)) = sigmoid(2 a)
+    return z * sigmoid_f32(1.59576912160573071f * fmaf(0.044715f * z * z, z, z));
+}
 __device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float dyn_tanh(const DynTanh& p, int n, float v) { return fmaf(tanhf(p.alpha * v), p.w[n], p.b[n]); }
 
@@ -96,7 +123,12 @@ template <typename A>
 __device__ __forceinline__ void linear_store(const Linear& l, int t, int n, float v)
 {
     switch (l.mode) {
-    case kLinF32: reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n] = v; break;
+    case kLinF32: reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n] = l.cap > 0.0f ? l.cap * tanhf(v / l.cap) : v; break;
+    case kLinGelu: reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(gelu_tanh_f32(v)); break;
+    case kLinLogDecay:
+        if (l.split && n >= l.split) reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n - l.split] = act_from<A>(v);
+        else l.dt[(size_t)t * l.ld_dt + n] = l.neg_exp_a[n] * softplus_f32(v + l.dt_bias[n]);
+        break;
     case kLinResidual: {
         float* px = l.x + (size_t)t * l.ld_x + n;
         const float r = *px + dyn_tanh(l.post, n, v);
@@ -104,14 +136,14 @@ __device__ __forceinline__ void linear_store(const Linear& l, int t, int n, floa
         if (l.next.w) reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(dyn_tanh(l.next, n, r));
         break;
     }
-    case kLinSsmIn:
+    case kLinMixerIn:
         if (n >= l.dt_row) {
-            l.dt[(size_t)t * l.ld_dt + n - l.dt_row] = softplus_f32(v + l.dt_bias[n - l.dt_row]);
+            l.dt[(size_t)t * l.ld_dt + n - l.dt_row] = l.dt_bias ? softplus_f32(v + l.dt_bias[n - l.dt_row]) : sigmoid_f32(v);
             break;
         }
-        if (l.conv.w && n >= l.conv_row) {
+        if (l.conv.w && n >= l.conv_row && n - l.conv_row < l.conv.channels) {
             const int c = n - l.conv_row, C = l.conv.channels;
-            float acc = l.conv.b[c];
+            float acc = l.conv.b ? l.conv.b[c] : 0.0f;
             for (int j = 0; j + 1 < l.conv.taps; j++) {
                 const float u = l.conv.tail[(size_t)j * C + c];
                 acc = fmaf(l.conv.w[(size_t)j * C + c], u, acc);

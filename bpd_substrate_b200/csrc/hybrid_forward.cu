@@ -1,19 +1,24 @@
-// Forward pass of the hybrid decoder: a list of layers, each with one of three mixers (retention, state-space duality,
-// latent attention) and an optional SwiGLU feed-forward, dynamic-tanh norms before and after every sublayer, the
-// embedding table as output head.
+// Forward pass of the hybrid decoders: a list of layers, each with one of five mixers (retention, state-space duality, gated delta
+// rule, latent or grouped-query attention) and an optional feed-forward (SwiGLU or GELU), around one of two residuals.
 //
-//   x = embed[token]
-//   x += norm1b(mixer(norm1(x)));  x += norm2b(ff(norm2(x)))          per layer
-//   logits = embed norm(x)
+// One stream, dynamic-tanh norms before and after every sublayer:
+//   x = embed[token];   x += norm1b(mixer(norm1(x)));  x += norm2b(ff(norm2(x)))  per layer;   logits = head norm(x)
+// Several streams joined by hyper-connections, RMS norms before every sublayer:
+//   x_s = scale embed[token];   y = sublayer(norm(sum_s in_s x_s)),  x_t <- sum_s mix_st x_s + out_t y;   logits = head norm(sum_s x_s)
 //
-// Norms have no launch of their own: the product that ends a sublayer adds to the residual through its post norm and
-// writes the next sublayer's normed input (linear.cu).  Launches per layer for one token: 4 (retention: in, recurrence,
-// gate + norm, out), 4 (state space: in with convolution and step sizes, recurrence, gate + norm, out), 7 (latent
-// attention), 2 (feed-forward).  One-token steps are recorded as a CUDA graph per sequence slot and replayed; token and
-// position are read from device memory.
+// Dynamic-tanh norms have no launch of their own: the product that ends a sublayer adds to the residual through its post norm
+// and writes the next sublayer's normed input (linear.cu).  With streams, a one-token step does the same with the streams in the
+// epilogue and the RMS norm in the product that follows; a prompt has one launch per sublayer for both (residual_streams.cu).
+// Launches per layer for one token: 4 (retention: in, recurrence, gate + norm, out), 4 (state space: in with convolution and step
+// sizes, recurrence, gate + norm, out), 4 (delta rule: in with convolutions and write shares, decays + gates, recurrence with gate
+// and norm, out), 7 (latent attention), 4 (grouped attention: in, norms + cache, attention, out), 2 (feed-forward).  One-token steps
+// are recorded as a CUDA graph per sequence slot and replayed; token and position are read from device memory.
 #include "decayed_scan.cuh"
+#include "delta_rule.cuh"
+#include "grouped_attention.cuh"
 #include "latent_attention.cuh"
 #include "launch.cuh"
+#include "residual_streams.cuh"
 #include "../../include/bpdq.h"
 
 #include <map>
@@ -57,8 +62,8 @@ struct Buffers {
     uint8_t* base = nullptr;
     size_t bytes = 0;
     int tokens = 0, context = 0, wanted = 0;
-    float *x, *dt, *partial, *logits;
-    void *h, *u, *o, *y, *xbc, *act, *cq, *q, *q_latent, *expanded, *rows;
+    float *x, *dt, *partial, *logits, *sum, *ys, *decays;
+    void *h, *u, *o, *y, *xbc, *act, *cq, *q, *q_latent, *expanded, *rows, *gates;
     int32_t *ids, *want;
     int* pos;
     long long* picked;
@@ -90,12 +95,29 @@ LatentShape latent_shape(const Plan& p, const bpdq_hybrid_layer& l)
     return s;
 }
 
+GroupedShape grouped_shape(const Plan& p, const bpdq_hybrid_layer& l)
+{
+    GroupedShape s = {};
+    s.heads = l.heads; s.groups = l.groups;
+    s.dim = l.key_dim; s.dim_pad = l.key_pad;
+    s.value_pad = l.value_pad;
+    s.chunk = l.chunk;
+    s.rows = l.cache_rows;
+    s.sink = 1;
+    s.scale = l.scale; s.cap = l.softcap;
+    s.eps = p.cfg.eps;
+    return s;
+}
+
 int in_rows(const bpdq_hybrid_layer& l)
 {
     if (l.mixer == BPDQ_MIX_RETENTION) return 2 * l.heads * l.key_pad + 2 * l.heads * l.value_pad;
     if (l.mixer == BPDQ_MIX_MAMBA2) return 2 * l.heads * l.value_pad + 2 * l.groups * l.key_pad + l.heads;
+    if (l.mixer == BPDQ_MIX_DELTA) return l.heads * l.value_pad + 2 * l.groups * l.key_pad + 2 * l.gate_rank_pad + l.heads;
+    if (l.mixer == BPDQ_MIX_GROUPED) return l.heads * l.key_pad + (l.kv_from < 0 ? l.groups * (l.key_pad + l.value_pad) : 0);
     return l.q_rank_pad + (l.kv_from < 0 ? l.kv_rank_pad + l.rot_pad : 0);
 }
+// (of a state-space or delta-rule layer)
 int conv_channels(const bpdq_hybrid_layer& l) { return l.heads * l.value_pad + 2 * l.groups * l.key_pad; }
 
 // Lays the buffers out (base == null: counts bytes).  A buffer is as large as the largest layer needs it.
@@ -103,7 +125,8 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
 {
     const size_t a = p.bf16_acts ? 2 : 4, t = (size_t)T;
     const int W = p.cfg.width_pad;
-    size_t u = 0, o = 0, xbc = 0, dt = 0, act = 0, cq = 0, q = 0, ql = 0, part = 0, exp = 0;
+    const bool streams = p.cfg.streams > 0;
+    size_t u = 0, o = 0, xbc = 0, dt = 0, act = 0, cq = 0, q = 0, ql = 0, part = 0, exp = 0, gates = 0, decays = 0;
     auto grow = [](size_t& m, size_t v) { if (v > m) m = v; };
     for (const auto& l : p.layers) {
         grow(u, t * ((in_rows(l) + 15) / 16 * 16));
@@ -112,6 +135,11 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
         if (l.mixer == BPDQ_MIX_MAMBA2) {
             grow(xbc, t * conv_channels(l));
             grow(dt, t * l.heads);
+        } else if (l.mixer == BPDQ_MIX_DELTA) {
+            grow(xbc, t * conv_channels(l));
+            grow(dt, t * l.heads);
+            grow(gates, t * l.heads * l.value_pad);
+            grow(decays, t * l.heads * l.key_pad);
         } else if (l.mixer == BPDQ_MIX_LATENT) {
             const LatentShape s = latent_shape(p, l);
             grow(cq, t * s.q_rank_pad);
@@ -127,7 +155,9 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
         at += (bytes + 255) / 256 * 256;
         return r;
     };
-    b.x = (float*)take(t * W * 4);
+    b.x = (float*)take(t * W * 4 * (streams ? p.cfg.streams : 1));
+    b.sum = (float*)take(streams && T == 1 ? t * W * 4 : 0);
+    b.ys = (float*)take(streams && T > 1 ? t * W * 4 : 0);
     b.h = take(t * W * a);
     b.u = take(u * a);
     b.o = take(o * a);
@@ -139,6 +169,8 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
     b.q_latent = take(ql * a);
     b.expanded = take(exp * a);
     b.rows = take((size_t)wanted * W * a);
+    b.gates = take(gates * a);
+    b.decays = (float*)take(decays * 4);
     b.dt = (float*)take(dt * 4);
     b.partial = (float*)take(part * 4);
     b.logits = (float*)take((size_t)wanted * p.cfg.vocab * 4);
@@ -194,21 +226,70 @@ struct Runner {
         l.mode = mode;
         return l;
     }
-    // the product that ends a sublayer: residual add through the post norm, then the next sublayer's normed input
-    int close(const uint16_t* W, int K, const void* in, const bpdq_dyn_tanh& post, const bpdq_dyn_tanh& next) const
+    // A sublayer's place in the residual: its norms, its connections, and what reads afterwards.
+    struct Sublayer {
+        const bpdq_dyn_tanh *norm, *post, *next;
+        const bpdq_stream_mix* mix;
+        const float* next_in;
+    };
+    // The product that begins a sublayer, on its normed input.  With streams one token's norm is part of it.
+    Linear open(const Sublayer& sub, const uint16_t* W, int N, void* out, int ld_out, int mode) const
     {
-        Linear l = product(W, p.cfg.width_pad, K, in, K, b.h, p.cfg.width_pad, kLinResidual);
+        Linear l = product(W, N, p.cfg.width_pad, b.h, p.cfg.width_pad, out, ld_out, mode);
+        if (p.cfg.streams && T == 1) {
+            l.in = b.sum;
+            l.norm_w = sub.norm->w;
+            l.norm_n = p.cfg.width;
+            l.norm_eps = p.cfg.eps;
+        }
+        return l;
+    }
+    // The product that ends a sublayer.  One stream: residual add through the post norm, then the next sublayer's normed
+    // input.  Several: into the streams, and what the next sublayer reads (of a prompt: normed).
+    int close(const Sublayer& sub, const uint16_t* W, int K, const void* in) const
+    {
+        const int Wp = p.cfg.width_pad;
+        Linear l = product(W, Wp, K, in, K, b.h, Wp, kLinResidual);
         l.x = b.x;
-        l.ld_x = p.cfg.width_pad;
-        l.post = norm_of(post);
-        l.next = norm_of(next);
-        return linear_forward(l, T, p.bf16_acts, s);
+        l.ld_x = Wp;
+        if (!p.cfg.streams) {
+            l.post = norm_of(*sub.post);
+            l.next = norm_of(*sub.next);
+            return linear_forward(l, T, p.bf16_acts, s);
+        }
+        if (T == 1) {
+            l.mode = kLinStreams;
+            l.streams = stream_mix(*sub.mix, p.cfg.streams, sub.next_in);
+            l.u = b.sum;
+            return linear_forward(l, T, p.bf16_acts, s);
+        }
+        l.mode = kLinF32;
+        l.out = b.ys;
+        const int rc = linear_forward(l, T, p.bf16_acts, s);
+        if (rc) return rc;
+        StreamStep st = streams_of(*sub.next);
+        st.y = b.ys;
+        st.m = stream_mix(*sub.mix, p.cfg.streams, sub.next_in);
+        return stream_step(st, T, p.bf16_acts, s);
+    }
+    // The streams, with `norm` ahead of what reads them.
+    StreamStep streams_of(const bpdq_dyn_tanh& norm) const
+    {
+        StreamStep st = {};
+        st.x = b.x;
+        st.norm_w = norm.w;
+        st.eps = p.cfg.eps;
+        st.width = p.cfg.width;
+        st.width_pad = p.cfg.width_pad;
+        if (T == 1) st.u = b.sum;
+        else st.h = b.h;
+        return st;
     }
 
-    int retention(const bpdq_hybrid_layer& l, const bpdq_dyn_tanh& next) const
+    int retention(const bpdq_hybrid_layer& l, const Sublayer& sub) const
     {
         const int HD = l.heads * l.key_pad, HV = l.heads * l.value_pad, N = in_rows(l);
-        int rc = linear_forward(product(l.w_in, N, p.cfg.width_pad, b.h, p.cfg.width_pad, b.u, N, kLinAct), T, p.bf16_acts, s);
+        int rc = linear_forward(open(sub, l.w_in, N, b.u, N, kLinAct), T, p.bf16_acts, s);
         if (rc) return rc;
         DecayedScan a = {};
         a.q = b.u; a.k = at(b.u, HD); a.v = at(b.u, 2 * HD);
@@ -227,13 +308,13 @@ struct Runner {
         if ((rc = gated_norm(b.o, HV, at(b.u, 2 * HD + HV), N, nullptr, b.y, HV, l.heads, l.value_dim, l.value_pad, l.heads, 0, p.cfg.eps, T,
                              p.bf16_acts, s)))
             return rc;
-        return close(l.w_o, HV, b.y, l.norm1b, next);
+        return close(sub, l.w_o, HV, b.y);
     }
 
-    int mamba2(const bpdq_hybrid_layer& l, const bpdq_dyn_tanh& next) const
+    int mamba2(const bpdq_hybrid_layer& l, const Sublayer& sub) const
     {
         const int HV = l.heads * l.value_pad, GN = l.groups * l.key_pad, C = conv_channels(l), N = in_rows(l), ld = (N + 15) / 16 * 16;
-        Linear in = product(l.w_in, N, p.cfg.width_pad, b.h, p.cfg.width_pad, b.u, ld, kLinSsmIn);
+        Linear in = open(sub, l.w_in, N, b.u, ld, kLinMixerIn);
         in.conv_row = HV;
         in.dt_row = HV + C;
         in.dt = b.dt;
@@ -256,57 +337,175 @@ struct Runner {
         if ((rc = decayed_scan(a, T, p.bf16_acts, s))) return rc;
         if ((rc = gated_norm(b.o, HV, b.u, ld, l.norm_w, b.y, HV, l.heads, l.value_dim, l.value_pad, l.norm_groups, 1, p.cfg.eps, T, p.bf16_acts, s)))
             return rc;
-        return close(l.w_o, HV, b.y, l.norm1b, next);
+        return close(sub, l.w_o, HV, b.y);
     }
 
-    int latent(const bpdq_hybrid_layer& l, const bpdq_dyn_tanh& next) const
+    int latent(const bpdq_hybrid_layer& l, const Sublayer& sub) const
     {
         const LatentShape sh = latent_shape(p, l);
         const bool own = l.kv_from < 0;
         const int N = in_rows(l);
         void* cache = state + (own ? l : p.layers[l.kv_from]).cache_offset;
-        int rc = linear_forward(product(l.w_in, N, p.cfg.width_pad, b.h, p.cfg.width_pad, b.u, N, kLinAct), T, p.bf16_acts, s);
+        int rc = linear_forward(open(sub, l.w_in, N, b.u, N, kLinAct), T, p.bf16_acts, s);
         if (rc) return rc;
         if ((rc = latent_prepare(sh, b.u, N, l.q_norm_w, l.kv_norm_w, b.cq, own ? cache : nullptr, b.pos, T, p.bf16_acts, s))) return rc;
         const int Q = sh.heads * sh.q_head();
         if ((rc = linear_forward(product(l.w_uq, Q, sh.q_rank_pad, b.cq, sh.q_rank_pad, b.q, Q, kLinAct), T, p.bf16_acts, s))) return rc;
         const LatentBuffers lb = {b.q_latent, b.partial, b.expanded};
         if ((rc = latent_attention(sh, b.q, reinterpret_cast<const bf16*>(l.w_ukv), cache, b.o, lb, b.pos, T, context, p.bf16_acts, s))) return rc;
-        return close(l.w_o, sh.heads * sh.value_pad, b.o, l.norm1b, next);
+        return close(sub, l.w_o, sh.heads * sh.value_pad, b.o);
+    }
+
+    // in rows: queries, keys, values (convolved), then what decays and gates are made of, then the write shares
+    int delta(const bpdq_hybrid_layer& l, const Sublayer& sub) const
+    {
+        const int HD = l.heads * l.key_pad, HV = l.heads * l.value_pad, GD = l.groups * l.key_pad, C = conv_channels(l), R = l.gate_rank_pad;
+        const int N = in_rows(l), ld = (N + 15) / 16 * 16;
+        Linear in = open(sub, l.w_in, N, b.u, ld, kLinMixerIn);
+        in.conv_row = 0;
+        in.dt_row = C + 2 * R;
+        in.dt = b.dt;
+        in.ld_dt = l.heads;
+        float* tail = (float*)(state + l.tail_offset);
+        if (T == 1) in.conv = ConvStep{l.conv_w, nullptr, tail, b.xbc, l.conv, C};
+        int rc = linear_forward(in, T, p.bf16_acts, s);
+        if (rc) return rc;
+        if (T > 1 && (rc = causal_conv(b.u, ld, b.xbc, C, l.conv, l.conv_w, nullptr, tail, T, p.bf16_acts, s))) return rc;
+        Linear d = product(l.w_gates, HD, R, at(b.u, C), ld, b.gates, HV, kLinLogDecay);
+        d.dt = b.decays;
+        d.ld_dt = HD;
+        d.dt_bias = l.dt_bias;
+        d.neg_exp_a = l.neg_exp_a;
+        if (T == 1) {           // decays and gates in one launch
+            d.N = HD + HV;
+            d.split = HD;
+            d.in2 = R;
+        } else if ((rc = linear_forward(product(l.w_gates + (size_t)HD * R, HV, R, at(b.u, C + R), ld, b.gates, HV, kLinAct), T, p.bf16_acts, s))) {
+            return rc;
+        }
+        if ((rc = linear_forward(d, T, p.bf16_acts, s))) return rc;
+        DeltaRule a = {};
+        a.q = b.xbc; a.k = at(b.xbc, GD); a.v = at(b.xbc, 2 * GD);
+        a.ld = C;
+        a.heads = l.heads; a.groups = l.groups;
+        a.key_pad = l.key_pad; a.value_dim = l.value_dim; a.value_pad = l.value_pad;
+        a.log_decay = b.decays;
+        a.beta = b.dt;
+        a.q_scale = l.scale;
+        a.unit_eps = 1e-6f;
+        a.state = (float*)(state + l.state_offset);
+        a.o = b.o;
+        const bool norms = T == 1 && delta_token_norms(l.key_pad, l.value_pad);
+        if (norms) {
+            a.norm_w = l.norm_w;
+            a.gate = b.gates;
+            a.eps = p.cfg.eps;
+        }
+        if ((rc = delta_rule(a, T, p.bf16_acts, s))) return rc;
+        if (!norms && (rc = gated_norm(b.o, HV, b.gates, HV, l.norm_w, b.y, HV, l.heads, l.value_dim, l.value_pad, l.heads, kNormWeightGate, p.cfg.eps, T,
+                                       p.bf16_acts, s)))
+            return rc;
+        return close(sub, l.w_o, HV, norms ? b.o : b.y);
+    }
+
+    int grouped(const bpdq_hybrid_layer& l, const Sublayer& sub) const
+    {
+        const GroupedShape sh = grouped_shape(p, l);
+        const bool own = l.kv_from < 0;
+        const int N = in_rows(l);
+        void* cache = state + (own ? l : p.layers[l.kv_from]).cache_offset;
+        int rc = linear_forward(open(sub, l.w_in, N, b.u, N, kLinAct), T, p.bf16_acts, s);
+        if (rc) return rc;
+        if ((rc = grouped_prepare(sh, b.u, N, own ? cache : nullptr, b.pos, T, p.bf16_acts, s))) return rc;
+        if ((rc = grouped_attention(sh, b.u, N, cache, b.o, b.pos, T, p.bf16_acts, s))) return rc;
+        return close(sub, l.w_o, l.heads * l.value_pad, b.o);
+    }
+
+    int mix(const bpdq_hybrid_layer& l, const Sublayer& sub) const
+    {
+        switch (l.mixer) {
+        case BPDQ_MIX_RETENTION: return retention(l, sub);
+        case BPDQ_MIX_MAMBA2: return mamba2(l, sub);
+        case BPDQ_MIX_DELTA: return delta(l, sub);
+        case BPDQ_MIX_GROUPED: return grouped(l, sub);
+        default: return latent(l, sub);
+        }
+    }
+
+    int feed_forward(const bpdq_hybrid_layer& l, const Sublayer& sub) const
+    {
+        const bool gelu = l.ff_kind == BPDQ_FF_GELU;
+        const int rc = linear_forward(open(sub, l.w_gate_up, gelu ? l.ff_pad : 2 * l.ff_pad, b.act, l.ff_pad, gelu ? kLinGelu : kLinSwiglu), T, p.bf16_acts, s);
+        return rc ? rc : close(sub, l.w_down, l.ff_pad, b.act);
+    }
+
+    int embed(const Sublayer& first) const
+    {
+        const int W = p.cfg.width_pad;
+        const bf16* table = reinterpret_cast<const bf16*>(p.cfg.embed);
+        if (p.cfg.streams) {
+            StreamStep st = streams_of(*first.norm);
+            st.table = table;
+            st.tokens = b.ids;
+            st.embed_scale = p.cfg.embed_scale;
+            st.vocab = p.cfg.vocab;
+            st.m.n = p.cfg.streams;
+            for (int i = 0; i < p.cfg.streams; i++) st.m.next[i] = first.next_in[i];
+            return stream_step(st, T, p.bf16_acts, s);
+        }
+        const DynTanh norm = norm_of(*first.norm);
+        return p.bf16_acts ? launch_ordered(k_embed_norm<bf16>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (bf16*)b.h, norm, W, p.cfg.vocab, device_error_flag())
+                           : launch_ordered(k_embed_norm<float>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (float*)b.h, norm, W, p.cfg.vocab, device_error_flag());
+    }
+
+    int copy_residual(float* out) const
+    {
+        if (p.cfg.streams) return stream_sum(b.x, p.cfg.streams, p.cfg.width, p.cfg.width_pad, out, T, s);
+        return check_cuda(cudaMemcpy2DAsync(out, (size_t)p.cfg.width * 4, b.x, (size_t)p.cfg.width_pad * 4, (size_t)p.cfg.width * 4, T,
+                                            cudaMemcpyDeviceToDevice, s));
     }
 
     int run(float* residuals, int n_want, bool all_wanted) const
     {
         const int W = p.cfg.width_pad, n = (int)p.layers.size();
-        const bf16* table = reinterpret_cast<const bf16*>(p.cfg.embed);
-        const DynTanh first = norm_of(n ? p.layers[0].norm1 : p.cfg.final_norm);
-        int rc = p.bf16_acts ? launch_ordered(k_embed_norm<bf16>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (bf16*)b.h, first, W, p.cfg.vocab, device_error_flag())
-                             : launch_ordered(k_embed_norm<float>, dim3((W + 1023) / 1024, T), 256, 0, s, table, (const int32_t*)b.ids, b.x, (float*)b.h, first, W, p.cfg.vocab, device_error_flag());
+        float ones[BPDQ_MAX_STREAMS];
+        for (float& v : ones) v = 1.0f;
+        Sublayer last = {&p.cfg.final_norm, nullptr, nullptr, nullptr, ones};       // the output head
+        auto mixer_of = [&](int i) {
+            if (i >= n) return last;
+            const bpdq_hybrid_layer& l = p.layers[i];
+            return Sublayer{&l.norm1, &l.norm1b, nullptr, &l.mix1, l.mix1.in};
+        };
+        auto follow = [](Sublayer& a, const Sublayer& next) { a.next = next.norm; a.next_in = next.next_in; };
+        // (a Sublayer's own reading weights are in next_in until the one that follows it is known)
+        int rc = embed(mixer_of(0));
         if (rc) return rc;
         for (int i = 0; i < n; i++) {
             const bpdq_hybrid_layer& l = p.layers[i];
-            const bpdq_dyn_tanh& after = i + 1 < n ? p.layers[i + 1].norm1 : p.cfg.final_norm;
-            const bpdq_dyn_tanh& next = l.ff_pad ? l.norm2 : after;
-            rc = l.mixer == BPDQ_MIX_RETENTION ? retention(l, next) : l.mixer == BPDQ_MIX_MAMBA2 ? mamba2(l, next) : latent(l, next);
-            if (rc) return rc;
+            Sublayer m = mixer_of(i), ff = {&l.norm2, &l.norm2b, nullptr, &l.mix2, l.mix2.in};
+            follow(m, l.ff_pad ? ff : mixer_of(i + 1));
+            if ((rc = mix(l, m))) return rc;
             if (l.ff_pad) {
-                if ((rc = linear_forward(product(l.w_gate_up, 2 * l.ff_pad, W, b.h, W, b.act, l.ff_pad, kLinSwiglu), T, p.bf16_acts, s))) return rc;
-                if ((rc = close(l.w_down, l.ff_pad, b.act, l.norm2b, after))) return rc;
+                follow(ff, mixer_of(i + 1));
+                if ((rc = feed_forward(l, ff))) return rc;
             }
-            if (residuals)
-                if ((rc = check_cuda(cudaMemcpy2DAsync(residuals + (size_t)i * T * p.cfg.width, (size_t)p.cfg.width * 4, b.x, (size_t)W * 4,
-                                                       (size_t)p.cfg.width * 4, T, cudaMemcpyDeviceToDevice, s))))
-                    return rc;
+            if (residuals && (rc = copy_residual(residuals + (size_t)i * T * p.cfg.width))) return rc;
         }
         if (n_want == 0) return 0;
+        const bool vec = p.cfg.streams && T == 1;       // the norm is part of the product; the same row for every place
         const void* rows = b.h;
-        if (!all_wanted) {
+        if (!all_wanted && !vec) {
             rc = p.bf16_acts ? launch_ordered(k_gather_rows<bf16>, grid_1d((long)n_want * W), 256, 0, s, (const bf16*)b.h, (const int32_t*)b.want, (bf16*)b.rows, W, n_want)
                              : launch_ordered(k_gather_rows<float>, grid_1d((long)n_want * W), 256, 0, s, (const float*)b.h, (const int32_t*)b.want, (float*)b.rows, W, n_want);
             if (rc) return rc;
             rows = b.rows;
         }
-        if ((rc = linear_forward(product(p.cfg.embed, p.cfg.vocab, W, rows, W, b.logits, p.cfg.vocab, kLinF32), n_want, p.bf16_acts, s))) return rc;
+        for (int i = 0; i < (vec ? n_want : 1); i++) {
+            Linear head = open(last, p.cfg.head, p.cfg.vocab, b.logits + (size_t)i * p.cfg.vocab, p.cfg.vocab, kLinF32);
+            if (!vec) head.in = rows;
+            head.cap = p.cfg.logit_cap;
+            if ((rc = linear_forward(head, vec ? 1 : n_want, p.bf16_acts, s))) return rc;
+        }
         return bpd_argmax_dim_cuda(b.logits, b.picked, n_want, p.cfg.vocab, 1, s);
     }
 };
@@ -334,8 +533,35 @@ int check_layer(const Plan& p, int i)
             const bpdq_hybrid_layer& o = p.layers[l.kv_from];
             return o.mixer == BPDQ_MIX_LATENT && o.kv_from < 0 && o.kv_rank == l.kv_rank && o.rot_dims == l.rot_dims ? 0 : BPDQ_ERR_ARG;
         }
+    case BPDQ_MIX_DELTA:
+        if (l.groups < 1 || l.heads % l.groups || l.conv < 1 || l.gate_rank_pad < 16 || l.gate_rank_pad % 16) return BPDQ_ERR_ARG;
+        if (!l.conv_w || !l.dt_bias || !l.neg_exp_a || !l.norm_w || !l.w_gates) return BPDQ_ERR_ARG;
+        return l.key_pad > 512 ? BPDQ_ERR_RANGE : 0;
+    case BPDQ_MIX_GROUPED: {
+        if (l.groups < 1 || l.heads % l.groups || l.chunk < 0 || l.cache_rows < 1 || l.softcap < 0.0f) return BPDQ_ERR_ARG;
+        if (l.kv_from < 0) return 0;
+        if (l.kv_from >= i) return BPDQ_ERR_ARG;
+        const bpdq_hybrid_layer& o = p.layers[l.kv_from];
+        return o.mixer == BPDQ_MIX_GROUPED && o.kv_from < 0 && o.groups == l.groups && o.key_dim == l.key_dim && o.value_dim == l.value_dim &&
+                       o.cache_rows == l.cache_rows ? 0 : BPDQ_ERR_ARG;
+    }
     default: return BPDQ_ERR_ARG;
     }
+}
+
+// Rows of a cache that are still needed by a portion's first token must not be those that its last token takes.
+int portion_limit(const Plan& p)
+{
+    int most = 65535;           // tokens are a grid dimension
+    for (const auto& l : p.layers)
+        if (l.mixer == BPDQ_MIX_GROUPED && l.chunk > 0 && l.cache_rows - l.chunk + 1 < most) most = l.cache_rows - l.chunk + 1;
+    return most < 1 ? 1 : most;
+}
+bool rows_suffice(const Plan& p, int pos, int T)
+{
+    for (const auto& l : p.layers)
+        if (l.mixer == BPDQ_MIX_GROUPED && pos + T > l.cache_rows && (l.chunk == 0 || T + l.chunk - 1 > l.cache_rows)) return false;
+    return true;
 }
 
 }  // namespace
@@ -348,7 +574,7 @@ extern "C" {
 
 void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers)
 {
-    if (!cfg || !cfg->embed || cfg->n_layers < 0 || (cfg->n_layers && !layers) || cfg->width < 1 || cfg->width_pad < cfg->width ||
+    if (!cfg || !cfg->embed || !cfg->head || cfg->streams < 0 || cfg->streams > BPDQ_MAX_STREAMS || cfg->logit_cap < 0.0f || cfg->n_layers < 0 || (cfg->n_layers && !layers) || cfg->width < 1 || cfg->width_pad < cfg->width ||
         cfg->width_pad % 16 || cfg->vocab < 1) {
         latch(BPDQ_ERR_ARG);
         return nullptr;
@@ -386,7 +612,7 @@ int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int 
     Plan* p = (Plan*)plan;
     cudaStream_t s = (cudaStream_t)stream;
     if (!p || !token_ids || n_tokens < 1 || pos < 0 || !state || n_want < 0 || (n_want && !want)) return latch(BPDQ_ERR_ARG);
-    if (n_tokens > 65535) return latch(BPDQ_ERR_RANGE);       // tokens are a grid dimension
+    if (n_tokens > 65535 || !rows_suffice(*p, pos, n_tokens)) return latch(BPDQ_ERR_RANGE);
     bool all = n_want == n_tokens;
     for (int i = 0; i < n_want; i++) {
         if (want[i] < 0 || want[i] >= n_tokens) return latch(BPDQ_ERR_RANGE);
@@ -430,6 +656,12 @@ int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int 
         return 0;
     }
     return check_cuda(cudaGraphLaunch(it->second, s));
+}
+
+int bpdq_hybrid_portion(void* plan)
+{
+    Plan* p = (Plan*)plan;
+    return p ? portion_limit(*p) : 0;
 }
 
 float* bpdq_hybrid_logits(void* plan)

@@ -1,7 +1,8 @@
-// Matrix products of the hybrid decoder: bf16 weights [N][K], activations bf16 or fp32, fp32 accumulation, and
-// everything elementwise that follows a product as its epilogue (residual add between two dynamic-tanh norms, SwiGLU
-// of paired rows, the step sizes and the one-token convolution of a state-space layer).  The dynamic-tanh norm needs
-// no row statistics, so no norm is a launch of its own.
+// Matrix products of the hybrid decoders: bf16 weights [N][K], activations bf16 or fp32, fp32 accumulation, and
+// everything elementwise that follows a product as its epilogue (residual add between two dynamic-tanh norms, residual
+// streams, SwiGLU of paired rows, GELU, step sizes, decays and the one-token convolution of a recurrent layer).  The
+// dynamic-tanh norm needs no row statistics; an RMS norm ahead of a one-token product is taken into the product, whose
+// CTAs all read the whole row anyway (the row enters times the norm's weight, the root mean square divides the sums).
 //
 //   k_linear_vec   one token: a warp streams two weight rows at a time with 16-byte loads, the first of them before the
 //                  launch ahead has finished (weights are constant); HBM bound
@@ -21,7 +22,8 @@ namespace bpdq {
 template <typename A>
 __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
 {
-    extern __shared__ float4 xs[];      // [2][K / 8]: first and second four of every eight activations
+    extern __shared__ float4 xs[];      // [2][K / 8]: first and second four of every eight activations (split: twice)
+    __shared__ float s_sum[8];
     constexpr int kBatch = 8;           // 16-byte loads in flight per row and lane
     const int units = l.K / 8, pairs = (l.N + 1) / 2;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -42,13 +44,41 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
     };
     if (p < pairs) fetch(0);
     pdl_wait();
-    const A* in = reinterpret_cast<const A*>(l.in);
-    for (int j = threadIdx.x; j < 2 * units; j += 256) xs[(j & 1) * units + (j >> 1)] = act_load4(in + 4 * j);
-    __syncthreads();
+    float rnorm = 1.0f;
+    if (l.norm_w) {
+        const float* in = reinterpret_cast<const float*>(l.in);
+        float sum = 0.0f;
+        for (int j = threadIdx.x; j < 2 * units; j += 256) {
+            float4 v = act_load4(in + 4 * j);
+            const float4 w4 = act_load4(l.norm_w + 4 * j);
+            sum = fmaf(v.x, v.x, sum); sum = fmaf(v.y, v.y, sum); sum = fmaf(v.z, v.z, sum); sum = fmaf(v.w, v.w, sum);
+            xs[(j & 1) * units + (j >> 1)] = make_float4(v.x * w4.x, v.y * w4.y, v.z * w4.z, v.w * w4.w);
+        }
+        sum = warp_sum(sum);
+        if (lane == 0) s_sum[warp] = sum;
+        __syncthreads();
+        sum = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) sum += s_sum[i];
+        rnorm = 1.0f / sqrtf(sum / (float)l.norm_n + l.norm_eps);
+    } else {
+        const A* in = reinterpret_cast<const A*>(l.in);
+        for (int j = threadIdx.x; j < 2 * units; j += 256) xs[(j & 1) * units + (j >> 1)] = act_load4(in + 4 * j);
+        if (l.split)
+            for (int j = threadIdx.x; j < 2 * units; j += 256) xs[(2 + (j & 1)) * units + (j >> 1)] = act_load4(in + l.in2 + 4 * j);
+        __syncthreads();
+    }
     bool have = true;
     for (; p < pairs; p += stride) {
         const int row = 2 * p + lane;
+        const float4* x = l.split && 2 * p >= l.split ? xs + 2 * units : xs;
         const bool residual = l.mode == kLinResidual && lane < 2 && row < l.N;
+        const bool streams = l.mode == kLinStreams && lane < 2 && row < l.N;
+        float xo[kMaxStreams];
+        if (streams) {
+#pragma unroll
+            for (int i = 0; i < kMaxStreams; i++) xo[i] = i < l.streams.n ? l.x[(size_t)i * l.ld_x + row] : 0.0f;
+        }
         float xr = 0, pw = 0, pb = 0, nw = 0, nb = 0;       // what the residual epilogue of row 2 p + lane needs, ahead of its use
         if (residual) {
             xr = l.x[row];
@@ -64,7 +94,7 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
             for (int i = 0; i < kBatch; i++) {
                 const int u = base + lane + 32 * i;
                 if (u >= units) break;
-                const float4 x0 = xs[u], x1 = xs[units + u];
+                const float4 x0 = x[u], x1 = x[units + u];
 #pragma unroll
                 for (int r = 0; r < 2; r++) {
                     const uint4 q = w[r][i];
@@ -81,14 +111,27 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
         }
         acc[0] = warp_sum(acc[0]);
         acc[1] = warp_sum(acc[1]);
-        const float v = lane ? acc[1] : acc[0];
+        const float v = (lane ? acc[1] : acc[0]) * rnorm;
         if (l.mode == kLinSwiglu) {
-            if (lane == 0) reinterpret_cast<A*>(l.out)[p] = act_from<A>(silu_f32(acc[0]) * acc[1]);
+            if (lane == 0) reinterpret_cast<A*>(l.out)[p] = act_from<A>(silu_f32(acc[0] * rnorm) * (acc[1] * rnorm));
+        } else if (streams) {
+            float u = 0.0f;
+#pragma unroll
+            for (int i = 0; i < kMaxStreams; i++) {
+                if (i >= l.streams.n) break;
+                float r = l.streams.out[i] * v;
+#pragma unroll
+                for (int j = 0; j < kMaxStreams; j++)
+                    if (j < l.streams.n) r = fmaf(l.streams.mix[j][i], xo[j], r);
+                l.x[(size_t)i * l.ld_x + row] = r;
+                u = fmaf(l.streams.next[i], r, u);
+            }
+            l.u[row] = u;
         } else if (residual) {
             const float r = xr + fmaf(tanhf(l.post.alpha * v), pw, pb);
             l.x[row] = r;
             if (l.next.w) reinterpret_cast<A*>(l.out)[row] = act_from<A>(fmaf(tanhf(l.next.alpha * r), nw, nb));
-        } else if (l.mode != kLinResidual && lane < 2 && row < l.N) {
+        } else if (l.mode != kLinResidual && l.mode != kLinStreams && lane < 2 && row < l.N) {
             linear_store<A>(l, 0, row, v);
         }
     }
@@ -283,9 +326,10 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                 pw = post.w[n]; pb = post.b[n];
                 if (next.w) { nw = next.w[n]; nb = next.b[n]; }
             }
-            // rows of this warp that are only rounded and stored
+            // rows of this warp that are only rounded and stored (after a GELU)
             const int n_end = (n - lane) + 32;
-            const bool plain_warp = !((l.N | l.ld_out) & 1) && (l.mode == kLinAct || (l.mode == kLinSsmIn && n_end <= l.dt_row && !l.conv.w));
+            const bool plain_warp = !((l.N | l.ld_out) & 1) &&
+                                    (l.mode == kLinAct || l.mode == kLinGelu || (l.mode == kLinMixerIn && n_end <= l.dt_row && !l.conv.w));
             for (int c0 = 0; c0 < kCols; c0 += 16) {
                 int v[16];
                 tmem_ld(ta + c0, v);
@@ -317,6 +361,9 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                         if (live && t < T) reinterpret_cast<bf16*>(l.out)[(size_t)t * l.ld_out + n / 2] = act_from<bf16>(silu_f32(g) * u);
                     }
                 } else if (plain_warp) {
+                    if (l.mode == kLinGelu)
+#pragma unroll
+                        for (int j = 0; j < 16; j++) v[j] = __float_as_int(gelu_tanh_f32(__int_as_float(v[j])));
                     // two neighbouring rows per store: the even lane finishes even tokens, the odd lane odd ones
 #pragma unroll
                     for (int j = 0; j < 16; j += 2) {
@@ -388,8 +435,10 @@ static int launch_tc5(const Linear& l, int T, cudaStream_t s)
 int linear_forward(const Linear& l, int T, bool act_bf16, cudaStream_t s)
 {
     if (l.K % 16 || l.K < 16 || l.N < 1 || T < 1 || l.ld_in % 8) return latch(BPDQ_ERR_ARG);
+    if (T > 1 && (l.norm_w || l.split || l.mode == kLinStreams)) return latch(BPDQ_ERR_ARG);
+    if (l.mode == kLinStreams && (l.streams.n < 1 || l.streams.n > kMaxStreams)) return latch(BPDQ_ERR_ARG);
     if (T == 1) {
-        const size_t smem = (size_t)l.K * 4;
+        const size_t smem = (size_t)l.K * (l.split ? 8 : 4);
         if (smem > 200 * 1024) return latch(BPDQ_ERR_RANGE);
         int rc = act_bf16 ? allow_smem<k_linear_vec<bf16>>(200 * 1024) : allow_smem<k_linear_vec<float>>(200 * 1024);
         if (rc) return rc;

@@ -1,7 +1,8 @@
 """Generation: sequences of a model in slots, prompts in portions, one token per step after that.
 
 A model brings ``state_parts()``, ``capacity``, ``vocab``, ``stream``, ``lib`` and
-``step(seq, tokens, want, logits)``; the engine is the same for every family.  A step runs one sequence:
+``step(seq, tokens, want, logits)``, and ``portion`` if a step takes no more tokens than that; the engine is
+the same for every family.  A step runs one sequence:
 the next portion of its prompt or its last token.  Live requests take turns.
 """
 from collections import deque
@@ -26,7 +27,7 @@ class Engine:
     def __init__(self, model, slots=1, portion=2048):
         if portion < 1:
             raise ValueError("a portion has at least one token")
-        self.model, self.portion = model, portion
+        self.model, self.portion = model, min(portion, getattr(model, "portion", portion))
         self.slots = SequenceSlots(model.lib, model.state_parts(), model.capacity, slots, model.stream)
         self.live = {}        # key -> Sequence
 

@@ -1,9 +1,10 @@
-"""Hybrid decoders: a list of layers of retention, state-space duality (Mamba-2) or latent attention,
-with dynamic-tanh norms around every sublayer and the embedding table as output head (Gurusun).
+"""Hybrid decoders: a list of layers whose mixers differ.  This file holds what their designs share and one of them: layers of
+retention, state-space duality (Mamba-2) or latent attention, with dynamic-tanh norms around every sublayer and the embedding
+table as output head (Gurusun).  vuzelix.py holds the other.
 
-``HybridSpec`` reads config.json, ``pack`` turns a checkpoint's tensors into what the kernels read (inner
-sizes padded to multiples of 16 with zero weights, products that share an input stacked, gate and up
-rows interleaved), ``DeviceHybrid`` uploads them and runs ``bpdq_hybrid_forward``.  There is no CPU path.
+A spec reads config.json (sizes and constants, checked), lists the checkpoint's tensors and what a sequence holds, and packs
+tensors into what the kernels read (inner sizes padded to multiples of 16 with zero weights, products that share an input
+stacked, gate and up rows interleaved); ``DeviceHybrid`` uploads them and runs ``bpdq_hybrid_forward``.  There is no CPU path.
 """
 import ctypes as C
 import json
@@ -15,7 +16,6 @@ from . import capi
 from .safetensors_load import SafetensorsFile, bf16_to_f32
 from .sequences import StatePart, lay_out
 
-ARCHITECTURES = ("Gurusun",)
 MIXERS = {"retention": capi.MIX_RETENTION, "mamba2": capi.MIX_MAMBA2, "latent_attention": capi.MIX_LATENT}
 
 
@@ -39,18 +39,35 @@ def _rotation(where, m, limit):
     return dims, float(rot["base"])
 
 
-class HybridSpec:
-    """Sizes and constants of a model, checked."""
+class DecoderSpec:
+    """What every design of a hybrid decoder has.  A subclass names its architecture, checks its layers, and brings
+    ``tensor_shapes``, ``state_parts``, ``pack_layer`` and ``pack_ends``."""
+    architecture = None
 
     def __init__(self, config):
         self.config = config
-        if config.get("architecture") not in ARCHITECTURES:
-            raise ValueError(f"architecture {config.get('architecture')!r} is not one of {ARCHITECTURES}")
+        if config.get("architecture") != self.architecture:
+            raise ValueError(f"architecture {config.get('architecture')!r} is not {self.architecture}")
         _positive("config", config, "vocab", "width")
         self.vocab, self.width = config["vocab"], config["width"]
         self.width_pad = pad16(self.width)
         self.eps = float(config["norm"]["eps"])
         self.layers = config["layers"]
+        self.check()
+
+    def read_shapes(self, shape):
+        """Sizes that only the checkpoint's tensors tell; shape(name) gives one."""
+
+    @classmethod
+    def from_folder(cls, folder):
+        with open(os.path.join(folder, "config.json")) as f:
+            return cls(json.load(f))
+
+
+class HybridSpec(DecoderSpec):
+    architecture = "Gurusun"
+
+    def check(self):
         for i, layer in enumerate(self.layers):
             where, kind, m = f"layer {i}", layer.get("type"), layer.get("mixer")
             if kind not in MIXERS:
@@ -82,11 +99,6 @@ class HybridSpec:
                 if mlp.get("kind") != "dense":
                     raise ValueError(f"{where}: unknown feed-forward {mlp.get('kind')!r}")
                 _positive(where, mlp, "ff")
-
-    @classmethod
-    def from_folder(cls, folder):
-        with open(os.path.join(folder, "config.json")) as f:
-            return cls(json.load(f))
 
     def state_parts(self, act_bf16):
         """What a sequence holds, layer by layer."""
@@ -132,6 +144,31 @@ class HybridSpec:
         norm("final.norm")
         return out
 
+    def pack_layer(self, i, get):
+        return pack_layer(self, i, get)
+
+    def pack_ends(self, get):
+        """Embedding, head and final norm; numbers of the model's descriptor."""
+        return Ends(_cols(get.bf16("embed"), self.width_pad), None, _norm(get, "final.norm", self.width_pad), {})
+
+    def synthetic_value(self, name, leaf, shape, rng):
+        """Random values of a tensor that is no matrix of a product, or None."""
+        if name == "embed":
+            return rng.standard_normal(shape, dtype=np.float32)
+        if leaf == "alpha":
+            return np.float32(0.5)
+        if name.endswith(".conv.b") or (leaf == "b" and "norm" in name):
+            return 0.05 * rng.standard_normal(shape, dtype=np.float32)
+        if leaf in ("D",) or "norm" in leaf:
+            return 1.0 + 0.1 * rng.standard_normal(shape, dtype=np.float32)
+        if leaf == "A_log":
+            return np.log(rng.uniform(1.0, 4.0, shape)).astype(np.float32)
+        if leaf == "dt_bias":
+            return rng.uniform(-4.0, -1.0, shape).astype(np.float32)
+        if leaf == "conv":
+            return (0.5 * rng.standard_normal(shape)).astype(np.float32)
+        return None
+
 
 # ---- packing: zero padding of inner sizes
 
@@ -163,19 +200,30 @@ def rotary_frequencies(dims, base):
 
 
 class Pack:
-    """Host arrays of one layer as the kernels read them: `mats` (uint16 bf16 bits), `vecs` (fp32), `ints`."""
+    """Host arrays of one layer as the kernels read them: `mats` (uint16 bf16 bits), `vecs` (fp32), `norms` (w, b or None, alpha),
+    `mixes` (capi.StreamMix), and the descriptor's numbers: `ints`, `floats`."""
 
     def __init__(self):
-        self.mats, self.vecs, self.ints, self.norms, self.scale = {}, {}, {}, {}, 1.0
+        self.mats, self.vecs, self.ints, self.norms, self.mixes, self.floats = {}, {}, {}, {}, {}, {"scale": 1.0}
+
+
+class Ends:
+    """What lies around the layers: bf16 bits of the embedding and the head (None: the embedding again), the final norm, and
+    further numbers of the descriptor."""
+
+    def __init__(self, embed, head, norm, numbers):
+        self.embed, self.head, self.norm, self.numbers = embed, head, norm, numbers
+
+
+def _vec(get, name, total):
+    v = np.zeros(total, np.float32)
+    a = get.f32(name)
+    v[:a.size] = a
+    return v
 
 
 def _norm(get, name, width_pad):
-    def vec(n):
-        v = np.zeros(width_pad, np.float32)
-        a = get.f32(n)
-        v[:a.size] = a
-        return v
-    return vec(name), vec(name + ".b"), float(get.f32(name + ".alpha").reshape(()))
+    return _vec(get, name, width_pad), _vec(get, name + ".b", width_pad), float(get.f32(name + ".alpha").reshape(()))
 
 
 def pack_layer(spec, i, get):
@@ -202,7 +250,7 @@ def pack_layer(spec, i, get):
         decay = np.asarray(m["decay"], np.float64)
         out.vecs.update(rot_freq=rotary_frequencies(dims, base), decay=decay, log_decay=np.log(decay))
         out.ints.update(rot_dims=dims)
-        out.scale = D ** -0.5
+        out.floats["scale"] = D ** -0.5
     elif kind == "mamba2":
         G = m["groups"]
         inner, gn, taps = H * V, G * D, m["conv"]
@@ -235,7 +283,7 @@ def pack_layer(spec, i, get):
         out.mats["w_ukv"] = np.concatenate([padded_rows("uk", rows_d, H * Dp, Rp), padded_rows("uv", rows_v, H * Vp, Rp)])
         out.vecs.update(q_norm_w=_spread(get.f32(p + "dq.norm"), 0, np.arange(Q), Qp), rot_freq=rotary_frequencies(r, m["rot"]["base"]))
         out.ints.update(rot_dims=r, rot_pad=rp, q_rank=Q, q_rank_pad=Qp, kv_rank=R, kv_rank_pad=Rp)
-        out.scale = float(m["scale"])
+        out.floats["scale"] = float(m["scale"])
     out.norms["norm1"] = _norm(get, f"l{i}.norm1", Wp)
     out.norms["norm1b"] = _norm(get, f"l{i}.norm1b", Wp)
     if layer.get("mlp"):
@@ -265,6 +313,9 @@ class ArrayTensors:
     def f32(self, name):
         return bf16_to_f32(self._bits[name])
 
+    def shape(self, name):
+        return self._bits[name].shape
+
 
 def synthetic_tensors(spec, seed=0):
     """Random weights of the right shapes (bf16 bits): products keep activations O(1)."""
@@ -282,25 +333,8 @@ def synthetic_tensors(spec, seed=0):
         return np.resize(np.roll(bits, start)[:pool.size - 7], shape)
 
     for name, shape in spec.tensor_shapes().items():
-        leaf = name.rsplit(".", 1)[-1]
-        if name == "embed":
-            v = rng.standard_normal(shape, dtype=np.float32)
-        elif leaf == "alpha":
-            v = np.float32(0.5)
-        elif name.endswith(".conv.b") or (leaf == "b" and "norm" in name):
-            v = 0.05 * rng.standard_normal(shape, dtype=np.float32)
-        elif leaf in ("D",) or "norm" in leaf:
-            v = 1.0 + 0.1 * rng.standard_normal(shape, dtype=np.float32)
-        elif leaf == "A_log":
-            v = np.log(rng.uniform(1.0, 4.0, shape)).astype(np.float32)
-        elif leaf == "dt_bias":
-            v = rng.uniform(-4.0, -1.0, shape).astype(np.float32)
-        elif leaf == "conv":
-            v = (0.5 * rng.standard_normal(shape)).astype(np.float32)
-        else:
-            out[name] = matrix(shape)
-            continue
-        out[name] = f32_to_bf16(np.asarray(v, np.float32))
+        v = spec.synthetic_value(name, name.rsplit(".", 1)[-1], shape, rng)
+        out[name] = matrix(shape) if v is None else f32_to_bf16(np.asarray(v, np.float32))
     return out
 
 
@@ -316,35 +350,40 @@ class DeviceHybrid:
         self._own_stream = stream is None
         self.stream = lib.bpdq_stream_create() if stream is None else stream
         self._allocs, self.weight_bytes = [], 0
+        spec.read_shapes(get.shape)
         self.parts = spec.state_parts(dtype == "bfloat16")
-        offsets = lay_out(self.parts, capacity).offsets
+        offsets, rows = lay_out(self.parts, capacity).offsets, {p.name: p.count(capacity) for p in self.parts}
         self.layers = (capi.HybridLayer * max(1, len(spec.layers)))()
         for i in range(len(spec.layers)):
-            pk, dst = pack_layer(spec, i, get), self.layers[i]
-            for k, v in pk.ints.items():
+            pk, dst = spec.pack_layer(i, get), self.layers[i]
+            for k, v in list(pk.ints.items()) + list(pk.floats.items()) + list(pk.mixes.items()):
                 setattr(dst, k, v)
             for k, v in pk.mats.items():
                 setattr(dst, k, self._up(np.ascontiguousarray(v, np.uint16)))
             for k, v in pk.vecs.items():
                 setattr(dst, k, self._up(np.ascontiguousarray(v, np.float32)))
             for k, (w, b, alpha) in pk.norms.items():
-                setattr(dst, k, capi.DynTanh(self._up(w), self._up(b), alpha))
-            dst.scale = pk.scale
+                setattr(dst, k, self._norm_of(w, b, alpha))
+            dst.cache_rows = rows.get(f"l{i if dst.kv_from < 0 else dst.kv_from}.cache", 0)
             for part in ("state", "tail", "cache"):
                 setattr(dst, part + "_offset", offsets.get(f"l{i}.{part}", 0))
-        w, b, alpha = _norm(get, "final.norm", spec.width_pad)
-        self.config = capi.HybridConfig(len(spec.layers), spec.width, spec.width_pad, spec.vocab, int(dtype == "bfloat16"), spec.eps,
-                                        self._up(_cols(get.bf16("embed"), spec.width_pad)), capi.DynTanh(self._up(w), self._up(b), alpha))
+        ends = spec.pack_ends(get)
+        self.config = capi.HybridConfig(n_layers=len(spec.layers), width=spec.width, width_pad=spec.width_pad, vocab=spec.vocab,
+                                        act_bf16=int(dtype == "bfloat16"), eps=spec.eps, final_norm=self._norm_of(*ends.norm), **ends.numbers)
+        self.config.embed = self._up(ends.embed)
+        self.config.head = self.config.embed if ends.head is None else self._up(ends.head)
         self.plan = lib.bpdq_hybrid_create(C.byref(self.config), self.layers)
         capi.check(lib.bpdq_last_status(), "hybrid decoder set-up")
         if not self.plan:
             raise capi.BpdqError("bpdq_hybrid_create refused the model")
+        self.portion = lib.bpdq_hybrid_portion(self.plan)       # most tokens of one step
 
     @classmethod
-    def from_folder(cls, folder, **kw):
-        spec = HybridSpec.from_folder(folder)
+    def from_folder(cls, folder, spec_class=HybridSpec, **kw):
+        spec = spec_class.from_folder(folder)
         f = SafetensorsFile(os.path.join(folder, "model.safetensors"))
         try:
+            spec.read_shapes(f.shape)
             for name, shape in spec.tensor_shapes().items():
                 got = tuple(f.tensors[name]["shape"]) if name in f else None
                 if got != tuple(shape):
@@ -363,6 +402,9 @@ class DeviceHybrid:
         self.weight_bytes += arr.nbytes
         return p
 
+    def _norm_of(self, w, b, alpha):
+        return capi.DynTanh(self._up(w), None if b is None else self._up(b), alpha)
+
     def state_parts(self):
         return self.parts
 
@@ -375,6 +417,8 @@ class DeviceHybrid:
             raise ValueError("a step needs at least one token")
         if seq.length + n > seq.capacity:
             raise ValueError(f"the sequence would hold {seq.length + n} tokens, its slot has room for {seq.capacity}")
+        if n > self.portion:
+            raise ValueError(f"a step of {n} tokens; this model takes up to {self.portion}")
         if tokens.min() < 0 or tokens.max() >= self.vocab:
             raise ValueError(f"token ids run from 0 to {self.vocab - 1}")
         capi.check(self.lib.bpdq_hybrid_forward(self.plan, tokens.ctypes.data, n, seq.length, seq.base, want.ctypes.data, want.size, residuals,

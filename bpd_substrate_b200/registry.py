@@ -3,10 +3,20 @@ import json
 import os
 
 
-def _hybrid(path, dtype, capacity):
+def _hybrid(spec_class, path, dtype, capacity):
     from . import capi
     from .hybrid import DeviceHybrid
-    return DeviceHybrid.from_folder(path, dtype=dtype, capacity=capacity, lib=capi.load(part="hybrid"))
+    return DeviceHybrid.from_folder(path, spec_class, dtype=dtype, capacity=capacity, lib=capi.load(part="hybrid"))
+
+
+def _gurusun(path, dtype, capacity):
+    from .hybrid import HybridSpec
+    return _hybrid(HybridSpec, path, dtype, capacity)
+
+
+def _vuzelix(path, dtype, capacity):
+    from .vuzelix import VuzelixSpec
+    return _hybrid(VuzelixSpec, path, dtype, capacity)
 
 
 def _llama(path, dtype, capacity):
@@ -17,7 +27,7 @@ def _llama(path, dtype, capacity):
 
 
 # architecture -> loader(path, dtype, capacity)
-FAMILIES = {"Gurusun": _hybrid, "llama": _llama}
+FAMILIES = {"Gurusun": _gurusun, "Vuzelix": _vuzelix, "llama": _llama}
 
 
 def architecture_of(path):

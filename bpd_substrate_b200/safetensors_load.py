@@ -46,6 +46,11 @@ class SafetensorsFile:
     def __contains__(self, name):
         return name in self.tensors
 
+    def shape(self, name):
+        if name not in self.tensors:
+            raise KeyError(f"{self.path}: no tensor {name}")
+        return tuple(self.tensors[name]["shape"])
+
     def raw(self, name):
         """The tensor as stored (bf16 as uint16)."""
         if name not in self.tensors:

@@ -1,8 +1,8 @@
 """What the sequences being generated hold on the device, for every model alike.
 
 A model lists its parts: ``rows`` parts grow with the sequence (a KV or latent cache, room for ``capacity``
-tokens) and ``fixed`` parts do not (recurrent states, convolution windows; zero at the start of a
-sequence).  :class:`SequenceSlots` owns one device block with a slot per live sequence; a slot that is
+tokens, or for the latest ``limit`` of them where no token looks further back) and ``fixed`` parts do not
+(recurrent states, convolution windows; zero at the start of a sequence).  :class:`SequenceSlots` owns one device block with a slot per live sequence; a slot that is
 given back is used again by the next sequence.
 """
 from dataclasses import dataclass
@@ -18,9 +18,14 @@ class StatePart:
     nbytes: int              # of one token for rows, of the whole part for fixed
     rows: bool = False
     zero: bool = True        # cleared when a sequence starts (cache rows that are never read before they are written need not be)
+    limit: int = 0           # most rows that are kept (token i in row i mod limit); 0: all
+
+    def count(self, capacity):
+        """Rows of the part in a slot."""
+        return (min(capacity, self.limit) if self.limit else capacity) if self.rows else 1
 
     def size(self, capacity):
-        n = self.nbytes * capacity if self.rows else self.nbytes
+        n = self.nbytes * self.count(capacity)
         return -(-n // ALIGN) * ALIGN
 
 

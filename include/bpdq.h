@@ -443,7 +443,8 @@ int bpd_llama_forward_ws_cuda(const int32_t* token_ids, int n_tokens, const bpd_
                               void* k_cache, void* v_cache, float* logits_out, long long* token_out, void* workspace,
                               size_t workspace_bytes, void* stream);
 
-/* ---- hybrid decoder: layers of retention, state-space duality (Mamba-2) or latent attention on bf16 weights ----
+/* ---- hybrid decoders: layers of retention, state-space duality (Mamba-2), a gated delta rule, latent or grouped-query
+ * attention on bf16 weights ----
  * Weights are bf16 [out][in]; activations bf16 or fp32 (act_bf16); residual stream, norms, scores, softmax, decays and
  * recurrent states are fp32.  Inner sizes are padded to multiples of 16 with zero weights (the *_pad fields).
  *
@@ -458,13 +459,13 @@ int bpd_decayed_scan_cuda(const void* q, int ld_q, const void* k, int ld_k, cons
 /* pairs (i, i + rot_dims / 2) of q and k turn by (pos + t) rot_freq[i], in place; then k *= k_scale */
 int bpd_rotate_half_qk_cuda(void* q, void* k, int ld, int n_tokens, int heads, int dim_pad, int rot_dims, const float* rot_freq, float k_scale,
                             const int32_t* pos, int act_bf16, void* stream);
-/* out = silu(b + sum_j w[j] in[t - taps + 1 + j]) per channel; tail [taps - 1][channels]: the inputs before token 0,
+/* out = silu(b + sum_j w[j] in[t - taps + 1 + j]) per channel (b NULL: 0); tail [taps - 1][channels]: the inputs before token 0,
  * oldest first, moved on to the last token */
 int bpd_causal_conv_silu_cuda(const void* in, int ld_in, void* out, int n_tokens, int channels, int taps, const float* w, const float* b, float* tail,
                               int act_bf16, void* stream);
-/* over `parts` equal parts: gate_first ? rms_norm(o silu(g)) w : rms_norm(o) silu(g) */
+/* over `parts` equal parts: form 0: rms_norm(o) silu(g), 1: rms_norm(o silu(g)) w, 2: rms_norm(o) w sigmoid(g) */
 int bpd_gated_norm_cuda(const void* o, int ld_o, const void* g, int ld_g, const float* w, void* y, int ld_y, int n_tokens, int heads, int value_dim,
-                        int value_pad, int parts, int gate_first, float eps, int act_bf16, void* stream);
+                        int value_pad, int parts, int form, float eps, int act_bf16, void* stream);
 typedef struct {
     int heads, dim_pad, value_pad, rank, rank_pad, rot_dims, rot_pad, q_rank, q_rank_pad;
     float scale, eps;
@@ -479,33 +480,70 @@ int bpd_latent_prepare_cuda(const bpdq_latent_shape* shape, const void* u, int l
 int bpd_latent_attention_cuda(const bpdq_latent_shape* shape, void* q, const uint16_t* w_ukv, const void* cache, void* o, const int32_t* pos,
                               int n_tokens, int context, int act_bf16, void* stream);
 
+/* Gated delta rule with a decay per key channel.  Per head and token, from and to state [heads][key_pad][value_pad]:
+ * S = diag(exp(log_decay)) S, u = beta (v - S^T k), S += k u^T, o = S^T q; k and q of unit length (x / sqrt(x.x + unit_eps)), q then
+ * times q_scale, both shared by heads / groups heads.  q, k, v rows are ld apart; log_decay [tokens][heads * key_pad], beta
+ * [tokens][heads].  norm_w (one token only; NULL: o as it is) [heads * value_pad]: o = rms_norm(o) norm_w sigmoid(gate) */
+int bpd_delta_rule_cuda(const void* q, const void* k, const void* v, int ld, const float* log_decay, const float* beta, float q_scale, float unit_eps,
+                        float* state, void* o, const float* norm_w, const void* gate, float eps, int n_tokens, int heads, int groups, int key_pad,
+                        int value_dim, int value_pad, int act_bf16, void* stream);
+/* Grouped-query attention.  A position sees itself and earlier ones, with chunk > 0 only those of its chunk (chunks counted from
+ * position 0); score = scale q.k, with cap > 0 then cap tanh(score / cap); sink: one more score of 0 without a value.
+ * Position i is cached in row i mod rows of [groups][dim_pad] keys, then [groups][value_pad] values. */
+typedef struct {
+    int heads, groups, dim, dim_pad, value_pad, chunk, rows, sink;
+    float scale, cap, eps;
+} bpdq_grouped_shape;
+/* u rows: queries [heads][dim_pad], with append also keys [groups][dim_pad] and values [groups][value_pad], which become the
+ * cache rows of *pos + t; queries (in place) and keys are divided by their root mean square first.  o [tokens][heads][value_pad] */
+int bpd_grouped_attention_cuda(const bpdq_grouped_shape* shape, void* u, int ld_u, void* cache, int append, void* o, const int32_t* pos, int n_tokens,
+                               int act_bf16, void* stream);
+/* Residual streams x [tokens][streams][width_pad] joined by hyper-connections: x_t = sum_s mix[s][t] x_s + out[t] y, all from the
+ * old streams; then u = sum_t in[t] x_t (fp32) and h = rms_norm(u) norm_w, each when given */
+#define BPDQ_MAX_STREAMS 8
+typedef struct {
+    float mix[BPDQ_MAX_STREAMS * BPDQ_MAX_STREAMS];   /* [from][to] */
+    float out[BPDQ_MAX_STREAMS], in[BPDQ_MAX_STREAMS];
+} bpdq_stream_mix;
+int bpd_stream_step_cuda(const float* y, float* x, const bpdq_stream_mix* mix, int streams, const float* norm_w, float eps, int n_tokens, int width,
+                         int width_pad, void* h, float* u, int act_bf16, void* stream);
+
 /* The whole model.  Descriptors are host memory holding device pointers. */
 typedef struct {
     const float *w, *b;      /* [width_pad] */
     float alpha;
-} bpdq_dyn_tanh;             /* tanh(alpha x) * w + b */
-enum { BPDQ_MIX_RETENTION = 0, BPDQ_MIX_MAMBA2 = 1, BPDQ_MIX_LATENT = 2 };
+} bpdq_dyn_tanh;             /* tanh(alpha x) * w + b; RMS norms use w alone */
+enum { BPDQ_MIX_RETENTION = 0, BPDQ_MIX_MAMBA2 = 1, BPDQ_MIX_LATENT = 2, BPDQ_MIX_DELTA = 3, BPDQ_MIX_GROUPED = 4 };
+enum { BPDQ_FF_SWIGLU = 0, BPDQ_FF_GELU = 1 };
 typedef struct {
     int mixer, heads, groups;
     int key_dim, key_pad, value_dim, value_pad;       /* key: dim, state or unrotated dim */
-    int rot_dims, rot_pad, conv, norm_groups, q_rank, q_rank_pad, kv_rank, kv_rank_pad, kv_from, ff_pad;   /* kv_from -1: own latents; ff_pad 0: none */
-    float scale;                                      /* retention: of k; latent attention: of the scores */
+    int rot_dims, rot_pad, conv, norm_groups, q_rank, q_rank_pad, kv_rank, kv_rank_pad, kv_from, ff_pad;   /* kv_from -1: own latents or keys; ff_pad 0: none */
+    int ff_kind, gate_rank_pad, chunk, cache_rows;    /* gate_rank_pad: delta rule, of decays and gates; cache_rows: grouped attention */
+    float scale, softcap;                             /* retention: of k; delta rule: of q; attention: of the scores */
     const float *rot_freq, *decay, *log_decay;
     const float *conv_w, *conv_b, *dt_bias, *neg_exp_a, *d_skip, *norm_w;    /* conv_w [taps][channels] */
     const float *q_norm_w, *kv_norm_w;
-    const uint16_t *w_in, *w_uq, *w_ukv, *w_o, *w_gate_up, *w_down;           /* gate and up rows alternate */
+    const uint16_t *w_in, *w_uq, *w_ukv, *w_o, *w_gate_up, *w_down;           /* gate and up rows alternate (GELU: up rows alone) */
+    const uint16_t* w_gates;                          /* delta rule: decay rows [heads * key_pad], then gate rows [heads * value_pad] */
     bpdq_dyn_tanh norm1, norm1b, norm2, norm2b;
+    bpdq_stream_mix mix1, mix2;                       /* with streams: around the mixer, around the feed-forward */
     size_t state_offset, tail_offset, cache_offset;   /* bytes into a sequence's state */
 } bpdq_hybrid_layer;
+/* streams 0: one residual stream, dynamic-tanh norms before (norm1, norm2) and after (norm1b, norm2b) every sublayer.
+ * streams > 0: residual streams that start as embed_scale times the embedding, RMS norms before every sublayer; the final norm reads
+ * the streams' sum. */
 typedef struct {
-    int n_layers, width, width_pad, vocab, act_bf16;
-    float eps;
-    const uint16_t* embed;                            /* [vocab][width_pad], also the output head */
+    int n_layers, width, width_pad, vocab, act_bf16, streams;
+    float eps, embed_scale, logit_cap;                /* logit_cap 0: logits as they are */
+    const uint16_t *embed, *head;                     /* [vocab][width_pad]; they may be the same */
     bpdq_dyn_tanh final_norm;
 } bpdq_hybrid_config;
 void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers);
 void bpdq_hybrid_destroy(void* plan);
-/* Runs n_tokens (up to 65535) tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
+/* The most tokens one call may bring: 65535, or less where a layer keeps only cache_rows rows. */
+int bpdq_hybrid_portion(void* plan);
+/* Runs n_tokens (up to bpdq_hybrid_portion) tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
  * memory.  Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
  * the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
  * one-token steps as a CUDA graph per state address. */
