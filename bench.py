@@ -509,18 +509,18 @@ def main():
                     help="N > 1 GPUs: 1 = one all-gather after the step's GEMVs (default); more = the gather is cut into "
                          "chunks of layers, each on a second stream under the next chunk's GEMVs (measured slower at 2 GPUs: "
                          "0.783 ms against 0.753 ms per step, the NCCL kernels compete with CTAs that fill every SM)")
-    ap.add_argument("--workload", default="mistral7b", choices=["mistral7b", "llama70b", "hybrid"],
+    ap.add_argument("--workload", default="mistral7b", choices=["mistral7b", "llama70b", "hybrid", "vuzelix"],
                     help="hybrid: prefill and decode of the hybrid decoder (Gurusun) beside the Q8_0 Llama of equal size, one JSON line "
-                         "per number (one GPU; --width); mistral7b: the benchmark (every rank a full layer set, weak scaling); llama70b: the "
+                         "per number (one GPU; --width); vuzelix: the same of the Vuzelix decoder beside Gurusun; mistral7b: the benchmark (every rank a full layer set, weak scaling); llama70b: the "
                          "70B-shaped model row-sharded over the ranks (80 layers + output head, strong scaling)")
-    ap.add_argument("--width", type=int, action="append", help="hybrid: model widths (default 2048 and 4096)")
+    ap.add_argument("--width", type=int, action="append", help="hybrid, vuzelix: model widths (default 2048 and 4096)")
     ap.add_argument("--tokens", type=int, default=1, help="activation rows per product (llama70b sweep: 1 and 8)")
     ap.add_argument("--layers", type=int, default=None,
                     help="layers resident (32 is the benchmark; fewer only for profiler captures)")
     args = ap.parse_args()
     if args.layers is None:
         args.layers = N_LAYERS if args.workload == "mistral7b" else 80
-    if args.workload == "hybrid":
+    if args.workload in ("hybrid", "vuzelix"):
         import measure
         from bpd_substrate_b200 import capi
         lib = capi.load()
@@ -529,7 +529,12 @@ def main():
         sampler.start()
         status = 0
         for width in args.width or (2048, 4096):
-            status |= measure.hybrid_throughput(lib, width, (512, 2048), 4096, steps=min(args.steps, 50), warmup=max(args.warmup, 3))
+            sizes = dict(prompt_tokens=(512, 2048), context=4096, steps=min(args.steps, 50), warmup=max(args.warmup, 3))
+            if args.workload == "vuzelix":
+                status |= measure.hybrid_throughput(lib, "vuzelix", width, **sizes)
+            status |= measure.hybrid_throughput(lib, "hybrid", width, **sizes)
+            if args.workload == "hybrid":
+                status |= measure.llama_throughput(lib, width, **sizes)
         print(json.dumps({"clocks": sampler.stop(), "status": status}), flush=True)
         sys.exit(1 if status else 0)
     if args.impl == "reference":

@@ -180,7 +180,6 @@ SIGNATURES = {
     "bpd_grouped_attention_cuda": (i32, [vp, vp, i32, vp, i32, vp, vp, i32, i32, vp]),
     "bpd_stream_step_cuda": (i32, [vp, vp, vp, i32, vp, f32, i32, i32, i32, vp, vp, i32, vp]),
     "bpdq_hybrid_create": (vp, [vp, vp]),
-    "bpdq_hybrid_portion": (i32, [vp]),
     "bpdq_hybrid_destroy": (None, [vp]),
     "bpdq_hybrid_forward": (i32, [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp]),
     "bpdq_hybrid_logits": (vp, [vp]),

@@ -550,13 +550,6 @@ int check_layer(const Plan& p, int i)
 }
 
 // Rows of a cache that are still needed by a portion's first token must not be those that its last token takes.
-int portion_limit(const Plan& p)
-{
-    int most = 65535;           // tokens are a grid dimension
-    for (const auto& l : p.layers)
-        if (l.mixer == BPDQ_MIX_GROUPED && l.chunk > 0 && l.cache_rows - l.chunk + 1 < most) most = l.cache_rows - l.chunk + 1;
-    return most < 1 ? 1 : most;
-}
 bool rows_suffice(const Plan& p, int pos, int T)
 {
     for (const auto& l : p.layers)
@@ -612,7 +605,7 @@ int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int 
     Plan* p = (Plan*)plan;
     cudaStream_t s = (cudaStream_t)stream;
     if (!p || !token_ids || n_tokens < 1 || pos < 0 || !state || n_want < 0 || (n_want && !want)) return latch(BPDQ_ERR_ARG);
-    if (n_tokens > 65535 || !rows_suffice(*p, pos, n_tokens)) return latch(BPDQ_ERR_RANGE);
+    if (n_tokens > 65535 || !rows_suffice(*p, pos, n_tokens)) return latch(BPDQ_ERR_RANGE);       // (tokens are a grid dimension)
     bool all = n_want == n_tokens;
     for (int i = 0; i < n_want; i++) {
         if (want[i] < 0 || want[i] >= n_tokens) return latch(BPDQ_ERR_RANGE);
@@ -656,12 +649,6 @@ int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int 
         return 0;
     }
     return check_cuda(cudaGraphLaunch(it->second, s));
-}
-
-int bpdq_hybrid_portion(void* plan)
-{
-    Plan* p = (Plan*)plan;
-    return p ? portion_limit(*p) : 0;
 }
 
 float* bpdq_hybrid_logits(void* plan)

@@ -16,6 +16,7 @@ from . import capi
 from .safetensors_load import SafetensorsFile, bf16_to_f32
 from .sequences import StatePart, lay_out
 
+MAX_TOKENS = 65535      # of one step
 MIXERS = {"retention": capi.MIX_RETENTION, "mamba2": capi.MIX_MAMBA2, "latent_attention": capi.MIX_LATENT}
 
 
@@ -43,6 +44,7 @@ class DecoderSpec:
     """What every design of a hybrid decoder has.  A subclass names its architecture, checks its layers, and brings
     ``tensor_shapes``, ``state_parts``, ``pack_layer`` and ``pack_ends``."""
     architecture = None
+    portion = None          # most tokens of a step once cache rows are used again
 
     def __init__(self, config):
         self.config = config
@@ -376,7 +378,8 @@ class DeviceHybrid:
         capi.check(lib.bpdq_last_status(), "hybrid decoder set-up")
         if not self.plan:
             raise capi.BpdqError("bpdq_hybrid_create refused the model")
-        self.portion = lib.bpdq_hybrid_portion(self.plan)       # most tokens of one step
+        # most tokens of one step: less where a layer keeps only its latest rows
+        self.portion = spec.portion if any(p.rows and p.count(capacity) < capacity for p in self.parts) else MAX_TOKENS
 
     @classmethod
     def from_folder(cls, folder, spec_class=HybridSpec, **kw):

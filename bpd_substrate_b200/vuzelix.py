@@ -9,7 +9,6 @@ from .hybrid import DecoderSpec, Ends, Pack, _blocks, _cols, _positive, _spread,
 from .sequences import StatePart
 
 MIXERS = {"channel_delta": capi.MIX_DELTA, "attention": capi.MIX_GROUPED}
-PORTION = 4096          # attention layers keep this many rows beyond a chunk, so that a step of as many tokens overwrites none it needs
 
 
 def _number(where, d, key, positive=False):
@@ -21,6 +20,7 @@ def _number(where, d, key, positive=False):
 
 class VuzelixSpec(DecoderSpec):
     architecture = "Vuzelix"
+    portion = 4096          # attention layers keep this many rows beyond a chunk: a step of as many tokens overwrites none it needs
 
     def check(self):
         c = self.config
@@ -100,7 +100,7 @@ class VuzelixSpec(DecoderSpec):
             elif m.get("kv_from") is None:
                 reach = max(u["mixer"]["mask"]["size"] for j, u in enumerate(self.layers)
                             if u["type"] == "attention" and i in (j, u["mixer"].get("kv_from")))
-                parts.append(StatePart(f"l{i}.cache", a * m["kv_heads"] * (D + V), rows=True, zero=False, limit=reach + PORTION))
+                parts.append(StatePart(f"l{i}.cache", a * m["kv_heads"] * (D + V), rows=True, zero=False, limit=reach + self.portion))
         return parts
 
     def pack_layer(self, i, get):

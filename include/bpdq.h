@@ -541,10 +541,8 @@ typedef struct {
 } bpdq_hybrid_config;
 void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers);
 void bpdq_hybrid_destroy(void* plan);
-/* The most tokens one call may bring: 65535, or less where a layer keeps only cache_rows rows. */
-int bpdq_hybrid_portion(void* plan);
-/* Runs n_tokens (up to bpdq_hybrid_portion) tokens (host ids) of one sequence that already holds `pos` tokens; `state` is the sequence's device
- * memory.  Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
+/* Runs n_tokens (up to 65535; once a sequence outgrows a layer's cache_rows, up to cache_rows - chunk + 1) tokens (host ids) of one
+ * sequence that already holds `pos` tokens; `state` is the sequence's device memory. Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
  * the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
  * one-token steps as a CUDA graph per state address. */
 int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int pos, void* state, const int32_t* want, int n_want,

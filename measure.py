@@ -6,8 +6,9 @@
     python measure.py --llama-prefill [LAYERS] [TOKENS]
                                                     # the same layers, a prefill: rows against re-tiled weights
     python measure.py --hybrid-once prefill|decode [WIDTH] [TOKENS] [CONTEXT]
-                                                    # a few steps of the hybrid decoder (decode: launch by launch): a
-                                                    # small case for a profiler
+    python measure.py --vuzelix-once prefill|decode [WIDTH] [TOKENS] [CONTEXT]
+                                                    # a few steps of a hybrid decoder (Gurusun, Vuzelix; decode: launch
+                                                    # by launch): a small case for a profiler
     python measure.py --q8-tiles [N K]
                                                     # Q8_0 many-token product on re-tiled weights (tcgen05)
                                                     # beside the row-layout kernel, 1..512 tokens
@@ -247,7 +248,7 @@ def llama_decode(lib, n_layers=4, steps=32):
     return 0 if status == 0 else 1
 
 
-# ---- hybrid decoder beside the Q8_0 Llama at equal width, depth and feed-forward
+# ---- hybrid decoders beside each other and the Q8_0 Llama at equal width, depth and weights of the feed-forward
 
 def hybrid_config(width, n_layers=4, vocab=32000):
     """Layers as a real model of that width might have them, every one with a feed-forward of 3.5 widths: retention,
@@ -267,9 +268,26 @@ def hybrid_config(width, n_layers=4, vocab=32000):
     return {"architecture": "Gurusun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
 
 
-def hybrid_device(lib, width, capacity, n_layers=4, dtype="bfloat16", use_graph=True):
-    from bpd_substrate_b200 import hybrid
-    spec = hybrid.HybridSpec(hybrid_config(width, n_layers))
+def vuzelix_config(width, n_layers=4, vocab=32000):
+    """Layers as a real model of that width might have them: delta rule and grouped attention in turn, every other attention layer on
+    the keys of the one before; a feed-forward with as many weights as the SwiGLU of 3.5 widths beside it."""
+    H = width // 128
+    kinds = [("channel_delta", {"heads": H, "kv_heads": H, "dim": 128, "vdim": 128, "conv": 4}),
+             ("attention", {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5 * 4, "softcap": 50.0, "mask": {"size": 8192}})]
+    layers = [{"type": kinds[i % 2][0], "mixer": dict(kinds[i % 2][1]), "mlp": {"kind": "dense", "ff": width * 21 // 4}} for i in range(n_layers)]
+    for i in range(3, n_layers, 4):
+        layers[i]["mixer"]["kv_from"] = i - 2
+    return {"architecture": "Vuzelix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "streams": 4,
+            "residual_mult": 0.5, "logit_softcap": 30.0, "layers": layers}
+
+
+def hybrid_device(lib, width, capacity, n_layers=4, dtype="bfloat16", use_graph=True, model="hybrid"):
+    from bpd_substrate_b200 import hybrid, vuzelix
+    if model == "vuzelix":
+        spec = vuzelix.VuzelixSpec(vuzelix_config(width, n_layers))
+        spec.ranks = {i: (128, 128) for i, la in enumerate(spec.layers) if la["type"] == "channel_delta"}
+    else:
+        spec = hybrid.HybridSpec(hybrid_config(width, n_layers))
     return hybrid.DeviceHybrid(spec, hybrid.ArrayTensors(hybrid.synthetic_tensors(spec, 1)), dtype=dtype, capacity=capacity, lib=lib,
                                use_graph=use_graph)
 
@@ -277,26 +295,36 @@ def hybrid_device(lib, width, capacity, n_layers=4, dtype="bfloat16", use_graph=
 def hybrid_flops(spec, tokens):
     """Multiply-adds of the products of a prompt from the start, times two (attention and recurrences included)."""
     W, f = spec.width, 0
-    for la in spec.layers:
+    for i, la in enumerate(spec.layers):
         m, H = la["mixer"], la["mixer"]["heads"]
         if la["type"] == "retention":
             f += 2 * H * (m["dim"] + m["vdim"]) * W + H * m["vdim"] * W + 2 * H * m["dim"] * m["vdim"]
         elif la["type"] == "mamba2":
             f += (2 * H * m["vdim"] + 2 * m["groups"] * m["state"] + H) * W + H * m["vdim"] * W + 2 * H * m["state"] * m["vdim"]
+        elif la["type"] == "channel_delta":
+            a, g = spec.ranks[i]
+            f += (2 * m["kv_heads"] * m["dim"] + 2 * H * m["vdim"] + a + g + H) * W + H * (a * m["dim"] + g * m["vdim"]) + 3 * H * m["dim"] * m["vdim"]
+        elif la["type"] == "attention":
+            own = m.get("kv_from") is None
+            f += (H * m["dim"] + (m["kv_heads"] * (m["dim"] + m["vdim"]) if own else 0) + H * m["vdim"]) * W
+            f += H * (m["dim"] + m["vdim"]) * (min(tokens, m["mask"]["size"]) + 1) // 2
         else:
             f += m["q_rank"] * (W + H * (m["dim"] + m["rot_dim"])) + H * m["vdim"] * W + H * (m["dim"] + m["vdim"]) * m["kv_rank"]
             f += 0 if m.get("kv_from") is not None else (m["kv_rank"] + m["rot_dim"]) * W
             f += H * (m["dim"] + m["rot_dim"] + m["vdim"]) * (tokens + 1) // 2
-        f += 3 * la["mlp"]["ff"] * W if la["mlp"] else 0
+        f += (2 if spec.architecture == "Vuzelix" else 3) * la["mlp"]["ff"] * W if la["mlp"] else 0
     return 2 * f * tokens
 
 
 def hybrid_bytes_per_token(model, context):
-    """What one decoded token must read and write: weights, states (both ways), cache rows of every attention layer."""
+    """What one decoded token must read and write: weights (of an embedding table with a head beside it only a row), states
+    (both ways), cache rows of every attention layer."""
     spec, n = model.spec, model.weight_bytes
+    if model.config.head != model.config.embed:
+        n -= 2 * spec.vocab * spec.width_pad
     rows = {p.name: p.nbytes for p in model.parts}
     for i, la in enumerate(spec.layers):
-        if la["type"] == "latent_attention":
+        if la["type"] in ("latent_attention", "attention"):
             j = la["mixer"].get("kv_from")
             n += context * rows[f"l{i if j is None else j}.cache"]
         else:
@@ -304,17 +332,7 @@ def hybrid_bytes_per_token(model, context):
     return n
 
 
-def hybrid_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, emit=print):
-    """Prefill and decode of the hybrid decoder and of the Llama of equal width: one JSON object per number."""
-    import ctypes as C
-    import time
-
-    from bpd_substrate_b200 import llama
-    from bpd_substrate_b200.engine import Engine
-    peak, n_layers = _peak(), 4
-    capacity = max(max(prompt_tokens), context + 2 * (steps + warmup) + 80)
-    rng = np.random.default_rng(0)
-    toks = rng.integers(0, 32000, capacity).astype(np.int32)
+def throughput_timer(lib):
     e0, e1 = lib.bpdq_event_create(), lib.bpdq_event_create()
 
     def timed(stream, fn, n, warm):
@@ -326,11 +344,26 @@ def hybrid_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, em
             fn()
         lib.bpdq_event_record(e1, stream)
         return lib.bpdq_event_elapsed_ms(e0, e1) / n
+    return timed
+
+
+def throughput_capacity(prompt_tokens, context, steps, warmup):
+    return max(max(prompt_tokens), context + 2 * (steps + warmup) + 80)
+
+
+def hybrid_throughput(lib, model, width, prompt_tokens, context, steps=20, warmup=3, emit=print):
+    """Prefill and decode of a hybrid decoder ("hybrid": Gurusun, "vuzelix"): one JSON object per number."""
+    import time
+
+    from bpd_substrate_b200.engine import Engine
+    peak, n_layers, timed = _peak(), 4, throughput_timer(lib)
+    capacity = throughput_capacity(prompt_tokens, context, steps, warmup)
+    toks = np.random.default_rng(0).integers(0, 32000, capacity).astype(np.int32)
 
     def line(**kw):
-        emit(json.dumps(dict(kw, width=width, layers=n_layers, status=lib.bpdq_last_status())), flush=True)
+        emit(json.dumps(dict(model=model, **kw, width=width, layers=n_layers, status=lib.bpdq_last_status())), flush=True)
 
-    m = hybrid_device(lib, width, capacity, n_layers)
+    m = hybrid_device(lib, width, capacity, n_layers, model=model)
     e = Engine(m, 1, portion=max(prompt_tokens))
     for T in prompt_tokens:
         seq = e.slots.acquire()
@@ -340,22 +373,35 @@ def hybrid_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, em
             m.launch(seq, toks[:T], [T - 1])
         ms = timed(m.stream, prompt, max(3, steps // 4), warmup)
         e.slots.release(seq)
-        line(model="hybrid", phase="prefill", tokens=T, ms=round(ms, 4), tokens_per_s=round(T / ms * 1e3),
-             tflops=round(hybrid_flops(m.spec, T) / ms / 1e9, 1))
+        line(phase="prefill", tokens=T, ms=round(ms, 4), tokens_per_s=round(T / ms * 1e3), tflops=round(hybrid_flops(m.spec, T) / ms / 1e9, 1))
     seq = e.slots.acquire()
     for at in range(0, context, max(prompt_tokens)):
         m.launch(seq, toks[at:min(context, at + max(prompt_tokens))])
     ms = timed(m.stream, lambda: m.launch(seq, toks[seq.length:seq.length + 1], [0]), steps, warmup)
     e.slots.release(seq)
     nbytes = hybrid_bytes_per_token(m, context)
-    line(model="hybrid", phase="decode", context=context, ms_per_token=round(ms, 4), tokens_per_s=round(1e3 / ms, 1), bytes_per_token=nbytes,
+    line(phase="decode", context=context, ms_per_token=round(ms, 4), tokens_per_s=round(1e3 / ms, 1), bytes_per_token=nbytes,
          gbs=round(nbytes / ms / 1e6, 1), pct_of_measured_peak=round(100 * nbytes / ms / 1e6 / peak, 1))
     t0 = time.perf_counter()
     e.generate([toks[:64].tolist()], 65)
     t1 = time.perf_counter()
-    line(model="hybrid", phase="engine end to end, 64 prompt + 65 new tokens", tokens_per_s=round(65 / (t1 - t0), 1))
+    line(phase="engine end to end, 64 prompt + 65 new tokens", tokens_per_s=round(65 / (t1 - t0), 1))
     e.close()
     m.close()
+    return lib.bpdq_last_status()
+
+
+def llama_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, emit=print):
+    """The same numbers of the Q8_0 Llama of equal width, depth and feed-forward."""
+    import ctypes as C
+
+    from bpd_substrate_b200 import llama
+    peak, n_layers, timed = _peak(), 4, throughput_timer(lib)
+    capacity = throughput_capacity(prompt_tokens, context, steps, warmup)
+    toks = np.random.default_rng(0).integers(0, 32000, capacity).astype(np.int32)
+
+    def line(**kw):
+        emit(json.dumps(dict(kw, width=width, layers=n_layers, status=lib.bpdq_last_status())), flush=True)
 
     H = width // 128
     cfg = llama.make_config(n_layers=n_layers, n_heads=H, n_kv_heads=H // 4, head_dim=128, ffn_dim=width * 7 // 2, vocab_size=32000, max_seq_len=capacity)
@@ -392,10 +438,10 @@ def hybrid_throughput(lib, width, prompt_tokens, context, steps=20, warmup=3, em
     return lib.bpdq_last_status()
 
 
-def hybrid_once(lib, phase, width=2048, tokens=1024, context=2048, repeats=2):
+def hybrid_once(lib, model, phase, width=2048, tokens=1024, context=2048, repeats=2):
     """`repeats` prompts, or one-token steps launched one kernel after the other: nothing else on the device."""
     from bpd_substrate_b200.engine import Engine
-    m = hybrid_device(lib, width, max(tokens, context + repeats + 1), use_graph=False)
+    m = hybrid_device(lib, width, max(tokens, context + repeats + 1), use_graph=False, model=model)
     e = Engine(m, 1, portion=4096)
     toks = np.random.default_rng(0).integers(0, 32000, max(tokens, context + repeats))
     if phase == "prefill":
@@ -406,7 +452,7 @@ def hybrid_once(lib, phase, width=2048, tokens=1024, context=2048, repeats=2):
         e.feed(0, toks[:context], [], logits=False)
         for i in range(repeats):
             e.feed(0, toks[context + i:context + i + 1], [0], logits=False)
-    print(json.dumps({"hybrid_once": phase, "width": width, "status": lib.bpdq_last_status()}))
+    print(json.dumps({f"{model}_once": phase, "width": width, "status": lib.bpdq_last_status()}))
     e.close()
     m.close()
     return 0
@@ -419,8 +465,8 @@ def main():
         return llama_decode(lib, *[int(v) for v in sys.argv[2:3]])
     if len(sys.argv) >= 2 and sys.argv[1] == "--llama-prefill":
         return llama_prefill(lib, *[int(v) for v in sys.argv[2:4]])
-    if len(sys.argv) >= 3 and sys.argv[1] == "--hybrid-once":
-        return hybrid_once(lib, sys.argv[2], *[int(v) for v in sys.argv[3:6]])
+    if len(sys.argv) >= 3 and sys.argv[1] in ("--hybrid-once", "--vuzelix-once"):
+        return hybrid_once(lib, sys.argv[1][2:-5], sys.argv[2], *[int(v) for v in sys.argv[3:6]])
     if len(sys.argv) >= 2 and sys.argv[1] == "--q8-tiles":
         return q8_tiles(lib, *[int(v) for v in sys.argv[2:4]])
     if len(sys.argv) >= 3 and sys.argv[1] == "--q8-tiles-once":
