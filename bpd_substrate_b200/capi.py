@@ -170,6 +170,7 @@ SIGNATURES = {
     "gpu_vecmat_q8_0": (None, [vp, vp, vp, i32, i32]),
     # hybrid decoder
     "bpd_linear_bf16_cuda": (i32, [vp, vp, vp, i32, i32, i32, i32, vp]),
+    "bpd_linear_map_cuda": (i32, [vp, vp, vp, i32, i32, i32, i32, vp, vp, f32, i32, vp]),
     "bpd_decayed_scan_cuda": (i32, [vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp]),
     "bpd_rotate_half_qk_cuda": (i32, [vp, vp, i32, i32, i32, i32, i32, vp, f32, vp, i32, vp]),
     "bpd_causal_conv_silu_cuda": (i32, [vp, i32, vp, i32, i32, i32, vp, vp, vp, i32, vp]),
@@ -274,6 +275,7 @@ class StreamMix(C.Structure):
 
 MIX_RETENTION, MIX_MAMBA2, MIX_LATENT, MIX_DELTA, MIX_GROUPED = range(5)
 FF_SWIGLU, FF_GELU = range(2)
+MAP_GELU, MAP_CAP, MAP_LOG_DECAY, MAP_SIGMOID = range(4)
 
 
 class HybridLayer(C.Structure):

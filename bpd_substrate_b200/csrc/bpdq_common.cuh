@@ -54,7 +54,7 @@ Tuning& tuning();
 // ends (a larger replacement is a new allocation; launches in flight and captured graphs that hold
 // the old address stay valid).  Growing is refused while the stream is being captured.
 enum ScratchKind { kScratchGemmActs = 0, kScratchTc5Acts, kScratchTc5Reduce, kScratchTilesActs, kScratchForward,
-                   kScratchQ4ktActs, kScratchQ4ktReduce, kScratchQ80Acts, kScratchLatent, kScratchKinds };
+                   kScratchQ4ktActs, kScratchQ4ktReduce, kScratchQ80Acts, kScratchLatent, kScratchDelta, kScratchKinds };
 struct Workspace {
     uint8_t* base;
     size_t bytes, used;

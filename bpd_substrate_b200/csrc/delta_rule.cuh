@@ -21,8 +21,10 @@ struct DeltaRule {
     const float* norm_w;
     const void* gate;
     float eps;
+    void* scratch;                      // delta_scratch_bytes() for long bf16 portions, else null
 };
 int delta_rule(const DeltaRule& a, int T, bool act_bf16, cudaStream_t s);
+size_t delta_scratch_bytes(int heads, int key_pad, int value_pad, int T, bool act_bf16);
 // Whether a one-token call takes norm and gate in.
 bool delta_token_norms(int key_pad, int value_pad);
 

@@ -63,7 +63,7 @@ struct Buffers {
     size_t bytes = 0;
     int tokens = 0, context = 0, wanted = 0;
     float *x, *dt, *partial, *logits, *sum, *ys, *decays;
-    void *h, *u, *o, *y, *xbc, *act, *cq, *q, *q_latent, *expanded, *rows, *gates;
+    void *h, *u, *o, *y, *xbc, *act, *cq, *q, *q_latent, *expanded, *rows, *gates, *chunks;
     int32_t *ids, *want;
     int* pos;
     long long* picked;
@@ -126,7 +126,7 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
     const size_t a = p.bf16_acts ? 2 : 4, t = (size_t)T;
     const int W = p.cfg.width_pad;
     const bool streams = p.cfg.streams > 0;
-    size_t u = 0, o = 0, xbc = 0, dt = 0, act = 0, cq = 0, q = 0, ql = 0, part = 0, exp = 0, gates = 0, decays = 0;
+    size_t u = 0, o = 0, xbc = 0, dt = 0, act = 0, cq = 0, q = 0, ql = 0, part = 0, exp = 0, gates = 0, decays = 0, chunks = 0;
     auto grow = [](size_t& m, size_t v) { if (v > m) m = v; };
     for (const auto& l : p.layers) {
         grow(u, t * ((in_rows(l) + 15) / 16 * 16));
@@ -140,6 +140,7 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
             grow(dt, t * l.heads);
             grow(gates, t * l.heads * l.value_pad);
             grow(decays, t * l.heads * l.key_pad);
+            grow(chunks, delta_scratch_bytes(l.heads, l.key_pad, l.value_pad, T, p.bf16_acts));
         } else if (l.mixer == BPDQ_MIX_LATENT) {
             const LatentShape s = latent_shape(p, l);
             grow(cq, t * s.q_rank_pad);
@@ -170,6 +171,7 @@ size_t lay_out(const Plan& p, Buffers& b, uint8_t* base, int T, int context, int
     b.expanded = take(exp * a);
     b.rows = take((size_t)wanted * W * a);
     b.gates = take(gates * a);
+    b.chunks = take(chunks);
     b.decays = (float*)take(decays * 4);
     b.dt = (float*)take(dt * 4);
     b.partial = (float*)take(part * 4);
@@ -395,6 +397,7 @@ struct Runner {
         a.unit_eps = 1e-6f;
         a.state = (float*)(state + l.state_offset);
         a.o = b.o;
+        a.scratch = b.chunks;
         const bool norms = T == 1 && delta_token_norms(l.key_pad, l.value_pad);
         if (norms) {
             a.norm_w = l.norm_w;

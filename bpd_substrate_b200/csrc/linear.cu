@@ -476,4 +476,38 @@ int bpd_linear_bf16_cuda(const uint16_t* W, const void* x, float* out, int n_tok
     return linear_forward(l, n_tokens, act_bf16 != 0, (cudaStream_t)stream);
 }
 
+// The same product followed by what a decoder's epilogues do to its sums (BPDQ_MAP_*).
+int bpd_linear_map_cuda(const uint16_t* W, const void* x, void* out, int n_tokens, int N, int K, int map, const float* bias, const float* rate, float cap,
+                        int act_bf16, void* stream)
+{
+    if (n_tokens < 0 || N < 1 || K < 16 || (n_tokens > 0 && (!W || !x || !out))) return latch(BPDQ_ERR_ARG);
+    if (((uintptr_t)W | (uintptr_t)x) & 15) return latch(BPDQ_ERR_ALIGN);
+    if (n_tokens == 0) return 0;
+    Linear l = {};
+    l.W = reinterpret_cast<const bf16*>(W);
+    l.in = x;
+    l.N = N; l.K = K; l.ld_in = K;
+    l.out = out;
+    l.ld_out = N;
+    l.dt = reinterpret_cast<float*>(out);
+    l.ld_dt = N;
+    l.dt_bias = bias;
+    l.neg_exp_a = rate;
+    switch (map) {
+    case BPDQ_MAP_GELU: l.mode = kLinGelu; break;
+    case BPDQ_MAP_CAP:
+        if (!(cap > 0.0f)) return latch(BPDQ_ERR_ARG);
+        l.mode = kLinF32;
+        l.cap = cap;
+        break;
+    case BPDQ_MAP_LOG_DECAY:
+        if (!bias || !rate) return latch(BPDQ_ERR_ARG);
+        l.mode = kLinLogDecay;
+        break;
+    case BPDQ_MAP_SIGMOID: l.mode = kLinMixerIn; l.dt_bias = nullptr; break;      // (rows from 0 on are write shares)
+    default: return latch(BPDQ_ERR_ARG);
+    }
+    return linear_forward(l, n_tokens, act_bf16 != 0, (cudaStream_t)stream);
+}
+
 }  // extern "C"

@@ -451,6 +451,11 @@ int bpd_llama_forward_ws_cuda(const int32_t* token_ids, int n_tokens, const bpd_
  * Single mechanisms (device pointers; act_bf16 chooses the type of the void* activations): */
 /* out[t][n] = sum_k W[n][k] x[t][k], fp32 results; K a multiple of 16 */
 int bpd_linear_bf16_cuda(const uint16_t* W, const void* x, float* out, int n_tokens, int N, int K, int act_bf16, void* stream);
+/* the same product, each sum v of row n mapped: gelu(v), tanh form, in the activation type; or in fp32 cap tanh(v / cap),
+ * rate[n] softplus(v + bias[n]), sigmoid(v) */
+enum { BPDQ_MAP_GELU = 0, BPDQ_MAP_CAP = 1, BPDQ_MAP_LOG_DECAY = 2, BPDQ_MAP_SIGMOID = 3 };
+int bpd_linear_map_cuda(const uint16_t* W, const void* x, void* out, int n_tokens, int N, int K, int map, const float* bias, const float* rate, float cap,
+                        int act_bf16, void* stream);
 /* Per head h and token t: S = decay S + (dt k) v^T, o = S^T q + d_skip v, from and to state [heads][key_pad][value_pad].
  * decay[h] (and its logarithm), or exp(neg_exp_a[h] dt) with dt [tokens][heads]; q and k shared by heads / groups heads */
 int bpd_decayed_scan_cuda(const void* q, int ld_q, const void* k, int ld_k, const void* v, int ld_v, const float* decay, const float* log_decay,
@@ -542,8 +547,8 @@ typedef struct {
 void* bpdq_hybrid_create(const bpdq_hybrid_config* cfg, const bpdq_hybrid_layer* layers);
 void bpdq_hybrid_destroy(void* plan);
 /* Runs n_tokens (up to 65535; once a sequence outgrows a layer's cache_rows, up to cache_rows - chunk + 1) tokens (host ids) of one
- * sequence that already holds `pos` tokens; `state` is the sequence's device memory. Logits and their argmax are computed at the n_want places of `want` (host, 0 .. n_tokens - 1) and stay in
- * the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
+ * sequence that already holds `pos` tokens; `state` is the sequence's device memory.  Logits and their argmax are computed at the
+ * n_want places of `want` (host, 0 .. n_tokens - 1) and stay in the plan's buffers until its next call.  residuals: device [n_layers][n_tokens][width] or NULL.  use_graph: replay
  * one-token steps as a CUDA graph per state address. */
 int bpdq_hybrid_forward(void* plan, const int32_t* token_ids, int n_tokens, int pos, void* state, const int32_t* want, int n_want,
                         float* residuals, int use_graph, void* stream);
