@@ -443,48 +443,79 @@ int rotate_half_qk(void* q, void* k, int ld, int heads, int dim_pad, int rot_dim
 
 constexpr int kConvTile = 32;      // tokens per thread
 
-// Thread = (channel, tile of tokens), the window in registers (kTaps > 0) or read again per token.
-template <typename A>
+// Thread = (NC neighbouring channels, tile of tokens), the window in registers (up to four taps) or read again per token.
+template <typename A, int NC>
 __global__ void __launch_bounds__(128) k_causal_conv(const A* in, int ld_in, A* out, int channels, int taps,
                                                      const float* __restrict__ w, const float* __restrict__ b, const float* tail, int T)
 {
+    struct alignas(NC * sizeof(A)) Group { A v[NC]; };
+    struct alignas(NC * 4) Floats { float v[NC]; };
     pdl_launch_dependents();
-    pdl_wait();
-    const int c = blockIdx.x * 128 + threadIdx.x;
+    const int c = NC * (blockIdx.x * 128 + threadIdx.x);
     if (c >= channels) return;
     const int t0 = blockIdx.y * kConvTile, t1 = t0 + kConvTile < T ? t0 + kConvTile : T;
-    const float bias = b ? b[c] : 0.0f;
-    auto input = [&](int t) -> float {      // t >= -(taps - 1)
-        return t >= 0 ? act_load(in + (size_t)t * ld_in + c) : tail[(size_t)(t + taps - 1) * channels + c];
+    auto floats = [&](const float* p) -> Floats { return *reinterpret_cast<const Floats*>(p + c); };
+    Floats bias = {};
+    if (b) bias = floats(b);
+    auto input = [&](int t) -> Floats {      // t >= -(taps - 1)
+        if (t < 0) return floats(tail + (size_t)(t + taps - 1) * channels);
+        const Group g = *reinterpret_cast<const Group*>(in + (size_t)t * ld_in + c);
+        Floats f;
+#pragma unroll
+        for (int i = 0; i < NC; i++) f.v[i] = act_load(&g.v[i]);
+        return f;
+    };
+    auto store = [&](int t, const Floats& f) {
+        Group g;
+#pragma unroll
+        for (int i = 0; i < NC; i++) g.v[i] = act_from<A>(silu_act<A>(f.v[i]));
+        *reinterpret_cast<Group*>(out + (size_t)t * channels + c) = g;
     };
     if (taps <= 4) {
-        float wv[4], win[4];
+        Floats wv[4], win[3];
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int jj = j - (4 - taps);      // the last tap is always slot 3
-            wv[j] = jj >= 0 ? w[(size_t)jj * channels + c] : 0.0f;
-            win[j] = (j < 3 && jj >= 0) ? input(t0 - 3 + j) : 0.0f;
+            wv[j] = Floats{};
+            if (jj >= 0) wv[j] = floats(w + (size_t)jj * channels);
+        }
+        pdl_wait();
+#pragma unroll
+        for (int j = 0; j < 3; j++) {
+            win[j] = Floats{};
+            if (j - (4 - taps) >= 0) win[j] = input(t0 - 3 + j);
         }
         for (int tb = t0; tb < t1; tb += 8) {
-            float x[8];
-#pragma unroll
-            for (int i = 0; i < 8; i++) x[i] = tb + i < t1 ? input(tb + i) : 0.0f;
+            Floats x[8];
 #pragma unroll
             for (int i = 0; i < 8; i++) {
-                float acc = bias;
-                acc = fmaf(wv[0], win[0], acc);
-                acc = fmaf(wv[1], win[1], acc);
-                acc = fmaf(wv[2], win[2], acc);
-                acc = fmaf(wv[3], x[i], acc);
-                if (tb + i < t1) out[(size_t)(tb + i) * channels + c] = act_from<A>(silu_f32(acc));
+                x[i] = Floats{};
+                if (tb + i < t1) x[i] = input(tb + i);
+            }
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                Floats acc = bias;
+#pragma unroll
+                for (int k = 0; k < NC; k++) {
+                    acc.v[k] = fmaf(wv[0].v[k], win[0].v[k], acc.v[k]);
+                    acc.v[k] = fmaf(wv[1].v[k], win[1].v[k], acc.v[k]);
+                    acc.v[k] = fmaf(wv[2].v[k], win[2].v[k], acc.v[k]);
+                    acc.v[k] = fmaf(wv[3].v[k], x[i].v[k], acc.v[k]);
+                }
+                if (tb + i < t1) store(tb + i, acc);
                 win[0] = win[1]; win[1] = win[2]; win[2] = x[i];
             }
         }
     } else {
+        pdl_wait();
         for (int t = t0; t < t1; t++) {
-            float acc = bias;
-            for (int j = 0; j < taps; j++) acc = fmaf(w[(size_t)j * channels + c], input(t - taps + 1 + j), acc);
-            out[(size_t)t * channels + c] = act_from<A>(silu_f32(acc));
+            Floats acc = bias;
+            for (int j = 0; j < taps; j++) {
+                const Floats x = input(t - taps + 1 + j), wj = floats(w + (size_t)j * channels);
+#pragma unroll
+                for (int k = 0; k < NC; k++) acc.v[k] = fmaf(wj.v[k], x.v[k], acc.v[k]);
+            }
+            store(t, acc);
         }
     }
 }
@@ -507,8 +538,10 @@ template <typename A>
 static int launch_conv(const void* in, int ld_in, void* out, int channels, int taps, const float* w, const float* b, float* tail,
                        int T, cudaStream_t s)
 {
-    int rc = launch_ordered(k_causal_conv<A>, dim3((channels + 127) / 128, (T + kConvTile - 1) / kConvTile), 128, 0, s, (const A*)in, ld_in,
-                            (A*)out, channels, taps, w, b, (const float*)tail, T);
+    const bool pairs = channels % 2 == 0 && ld_in % 2 == 0 && !(((uintptr_t)in | (uintptr_t)out) % (2 * sizeof(A)));
+    const dim3 grid((channels / (pairs ? 2 : 1) + 127) / 128, (T + kConvTile - 1) / kConvTile);
+    int rc = pairs ? launch_ordered(k_causal_conv<A, 2>, grid, 128, 0, s, (const A*)in, ld_in, (A*)out, channels, taps, w, b, (const float*)tail, T)
+                   : launch_ordered(k_causal_conv<A, 1>, grid, 128, 0, s, (const A*)in, ld_in, (A*)out, channels, taps, w, b, (const float*)tail, T);
     if (rc || taps < 2) return rc;
     return launch_ordered(k_conv_tail<A>, (channels + 127) / 128, 128, 0, s, (const A*)in, ld_in, channels, taps, tail, T);
 }
@@ -523,7 +556,7 @@ int causal_conv(const void* in, int ld_in, void* out, int channels, int taps, co
 // ------------------------------------------------------------------ gate and norm
 
 // What multiplies: silu, or (after a norm with a weight) sigmoid of the gate.
-__device__ __forceinline__ float gate_value(int form, float g) { return form == kNormWeightGate ? sigmoid_f32(g) : silu_f32(g); }
+template <typename A> __device__ __forceinline__ float gate_value(int form, float g) { return form == kNormWeightGate ? sigmoid_act<A>(g) : silu_act<A>(g); }
 
 // Any sizes: one CTA per (part, token).  Values are kept in registers up to 16 per thread, else computed again.
 template <typename A>
@@ -562,7 +595,7 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
         }
 #pragma unroll
         for (int j = 0; j < kKeep; j++) {
-            gate[j] = gate_value(form, gate[j]);
+            gate[j] = gate_value<A>(form, gate[j]);
             if (form == kGateThenNorm) keep[j] *= gate[j];
             sum = fmaf(keep[j], keep[j], sum);
         }
@@ -570,7 +603,7 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
         for (int i = threadIdx.x; i < part; i += n) {
             const int c = where(i);
             float v = act_load(po + c);
-            if (form == kGateThenNorm) v *= silu_f32(act_load(pg + c));
+            if (form == kGateThenNorm) v *= silu_act<A>(act_load(pg + c));
             sum = fmaf(v, v, sum);
         }
     }
@@ -593,7 +626,7 @@ __global__ void __launch_bounds__(256) k_gated_norm(const A* o, int ld_o, const 
     } else {
         for (int i = threadIdx.x; i < part; i += n) {
             const int c = where(i);
-            const float v = act_load(po + c), z = gate_value(form, act_load(pg + c));
+            const float v = act_load(po + c), z = gate_value<A>(form, act_load(pg + c));
             py[c] = act_from<A>(v * z * scale * (form != kNormThenGate ? w[c] : 1.0f));
         }
     }
@@ -624,7 +657,7 @@ __global__ void __launch_bounds__(256) k_gated_norm_vec(const A* o, int ld_o, co
     float sum = 0.0f;
 #pragma unroll
     for (int j = 0; j < NJ; j++) {
-        z[j] = make_float4(gate_value(form, z[j].x), gate_value(form, z[j].y), gate_value(form, z[j].z), gate_value(form, z[j].w));
+        z[j] = make_float4(gate_value<A>(form, z[j].x), gate_value<A>(form, z[j].y), gate_value<A>(form, z[j].z), gate_value<A>(form, z[j].w));
         if (form == kGateThenNorm) v[j] = make_float4(v[j].x * z[j].x, v[j].y * z[j].y, v[j].z * z[j].z, v[j].w * z[j].w);
         sum = fmaf(v[j].x, v[j].x, sum); sum = fmaf(v[j].y, v[j].y, sum); sum = fmaf(v[j].z, v[j].z, sum); sum = fmaf(v[j].w, v[j].w, sum);
     }

@@ -108,14 +108,45 @@ __device__ __forceinline__ void act_store4(bf16* p, float4 v)
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 
-__device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float ex2(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float gelu_tanh_f32(float z)
+__device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+
+// Of results that are rounded to A: with bf16 activations a few units in the last place of fp32 do not matter.
+template <typename A> __device__ __forceinline__ float sigmoid_act(float z)
+{
+    if (sizeof(A) == 4) return sigmoid_f32(z);
+    return __fdividef(1.0f, 1.0f + ex2(-1.44269504088896341f * z));
+}
+template <typename A> __device__ __forceinline__ float silu_act(float z)
+{
+    if (sizeof(A) == 4) return z / (1.0f + expf(-z));
+    return z * sigmoid_act<A>(z);
+}
+template <typename A> __device__ __forceinline__ float gelu_act(float z)
 {
     // 0.5 (1 + tanh(a)) = sigmoid(2 a)
-    return z * sigmoid_f32(1.59576912160573071f * fmaf(0.044715f * z * z, z, z));
+    return z * sigmoid_act<A>(1.59576912160573071f * fmaf(0.044715f * z * z, z, z));
 }
-__device__ __forceinline__ float softplus_f32(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+// log(1 + e^z) = max(z, 0) + log(1 + e), e = e^-|z| <= 1; with fp32 activations by CUDA's functions, else by
+// log(1 + e) = 2 artanh(t), t = e / (2 + e) <= 1/3, whose Taylor series keeps the relative accuracy of small values.
+template <typename A> __device__ __forceinline__ float softplus_act(float z)
+{
+    if (sizeof(A) == 4) return softplus_f32(z);
+    const float e = ex2(-1.44269504088896341f * fabsf(z)), t = __fdividef(e, 2.0f + e), s = t * t;
+    float p = fmaf(s, 1.0f / 15, 1.0f / 13);
+    p = fmaf(s, p, 1.0f / 11);
+    p = fmaf(s, p, 1.0f / 9);
+    p = fmaf(s, p, 1.0f / 7);
+    p = fmaf(s, p, 1.0f / 5);
+    p = fmaf(s, p, 1.0f / 3);
+    return fmaxf(z, 0.0f) + 2.0f * fmaf(t * s, p, t);
+}
 __device__ __forceinline__ float dyn_tanh(const DynTanh& p, int n, float v) { return fmaf(tanhf(p.alpha * v), p.w[n], p.b[n]); }
 
 // Everything but the pairwise mode: row n, token t.
@@ -124,10 +155,10 @@ __device__ __forceinline__ void linear_store(const Linear& l, int t, int n, floa
 {
     switch (l.mode) {
     case kLinF32: reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n] = l.cap > 0.0f ? l.cap * tanhf(v / l.cap) : v; break;
-    case kLinGelu: reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(gelu_tanh_f32(v)); break;
+    case kLinGelu: reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(gelu_act<A>(v)); break;
     case kLinLogDecay:
         if (l.split && n >= l.split) reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n - l.split] = act_from<A>(v);
-        else l.dt[(size_t)t * l.ld_dt + n] = l.neg_exp_a[n] * softplus_f32(v + l.dt_bias[n]);
+        else l.dt[(size_t)t * l.ld_dt + n] = l.neg_exp_a[n] * softplus_act<A>(v + l.dt_bias[n]);
         break;
     case kLinResidual: {
         float* px = l.x + (size_t)t * l.ld_x + n;
@@ -154,7 +185,7 @@ __device__ __forceinline__ void linear_store(const Linear& l, int t, int n, floa
             const int last = l.conv.taps - 1;
             acc = fmaf(l.conv.w[(size_t)last * C + c], u, acc);
             if (last > 0) l.conv.tail[(size_t)(last - 1) * C + c] = u;
-            reinterpret_cast<A*>(l.conv.out)[c] = act_from<A>(silu_f32(acc));
+            reinterpret_cast<A*>(l.conv.out)[c] = act_from<A>(silu_act<A>(acc));
             break;
         }
         reinterpret_cast<A*>(l.out)[(size_t)t * l.ld_out + n] = act_from<A>(v);

@@ -130,8 +130,8 @@ __global__ void __launch_bounds__(256) k_delta_token(DeltaRule a)
             for (uint32_t i = 0; i < parts; i++) ss += s_part[i];
         }
         const float f = 1.0f / sqrtf(ss / (float)a.value_dim + a.eps);
-        o = make_float4(o.x * f * nw.x * sigmoid_f32(gate.x), o.y * f * nw.y * sigmoid_f32(gate.y), o.z * f * nw.z * sigmoid_f32(gate.z),
-                        o.w * f * nw.w * sigmoid_f32(gate.w));
+        o = make_float4(o.x * f * nw.x * sigmoid_act<A>(gate.x), o.y * f * nw.y * sigmoid_act<A>(gate.y), o.z * f * nw.z * sigmoid_act<A>(gate.z),
+                        o.w * f * nw.w * sigmoid_act<A>(gate.w));
     }
     if (phase == 0 && live) act_store4(reinterpret_cast<A*>(a.o) + at, o);
 }

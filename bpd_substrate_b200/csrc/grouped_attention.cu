@@ -65,13 +65,6 @@ int grouped_prepare(const GroupedShape& p, void* u, int ld_u, void* cache, const
 
 // ------------------------------------------------------------------ scores
 
-__device__ __forceinline__ float ex2(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 // Score in units of log2: tanh(z) = 1 - 2 / (1 + e^(2 z)), whose absolute error of an fp32 unit is all a capped score needs.
 struct ScoreMap {
     float plain, in, out;       // cap == 0: s plain;  else out tanh(s in / (2 log2 e))

@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(256, 2) k_linear_vec(Linear l)
         acc[1] = warp_sum(acc[1]);
         const float v = (lane ? acc[1] : acc[0]) * rnorm;
         if (l.mode == kLinSwiglu) {
-            if (lane == 0) reinterpret_cast<A*>(l.out)[p] = act_from<A>(silu_f32(acc[0] * rnorm) * (acc[1] * rnorm));
+            if (lane == 0) reinterpret_cast<A*>(l.out)[p] = act_from<A>(silu_act<A>(acc[0] * rnorm) * (acc[1] * rnorm));
         } else if (streams) {
             float u = 0.0f;
 #pragma unroll
@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(256) k_linear_tile(Linear l, int T)
 #pragma unroll
             for (int i = 0; i < 4; i += 2) {
                 const int n = n0 + 4 * tr + i;
-                if (n < l.N) reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n / 2] = silu_f32(acc[j][i]) * acc[j][i + 1];
+                if (n < l.N) reinterpret_cast<float*>(l.out)[(size_t)t * l.ld_out + n / 2] = silu_act<float>(acc[j][i]) * acc[j][i + 1];
             }
         } else {
 #pragma unroll
@@ -358,12 +358,12 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                         const float other = __shfl_xor_sync(0xFFFFFFFFu, __int_as_float((lane & 1) ? v[j] : v[j + 1]), 1);
                         const float g = (lane & 1) ? other : keep, u = (lane & 1) ? keep : other;
                         const int t = t0 + j + (lane & 1);
-                        if (live && t < T) reinterpret_cast<bf16*>(l.out)[(size_t)t * l.ld_out + n / 2] = act_from<bf16>(silu_f32(g) * u);
+                        if (live && t < T) reinterpret_cast<bf16*>(l.out)[(size_t)t * l.ld_out + n / 2] = act_from<bf16>(silu_act<bf16>(g) * u);
                     }
                 } else if (plain_warp) {
                     if (l.mode == kLinGelu)
 #pragma unroll
-                        for (int j = 0; j < 16; j++) v[j] = __float_as_int(gelu_tanh_f32(__int_as_float(v[j])));
+                        for (int j = 0; j < 16; j++) v[j] = __float_as_int(gelu_act<bf16>(__int_as_float(v[j])));
                     // two neighbouring rows per store: the even lane finishes even tokens, the odd lane odd ones
 #pragma unroll
                     for (int j = 0; j < 16; j += 2) {

@@ -41,8 +41,8 @@ def test_mapped_products(lib, bf16, T, N, K):
         got = (act.read(do) if kind == capi.MAP_GELU else do.read(np.float32)).reshape(T, N)
         assert normwise(got, want) < (act.tol if kind == capi.MAP_GELU else fine), kind
         if kind == capi.MAP_LOG_DECAY:             # small decays are exact in themselves, not only beside large ones
-            small = np.abs(want) < 0.05
-            assert np.max(np.abs(got[small] / want[small] - 1), initial=0) < 2e-4
+            small = (np.abs(want) < 0.05) & (np.abs(want) > 1e-7)
+            assert small.any() and np.max(np.abs(got[small] / want[small] - 1)) < 2e-4
 
 
 # ------------------------------------------------------------------ gated delta rule
@@ -169,16 +169,15 @@ def attention_case(lib, bf16, T, pos, H, G, D, V, chunk, rows=None, seed=0, sink
     Dp, Vp, L, eps = pad16(D), pad16(V), pos + T, 0.001
     rows, scale = rows or L + 5, 24.0 / D
     q, k, v = (act.host(rng.standard_normal(s)) for s in ((L, H, D), (L, G, D), (L, G, V)))
-    aims = 0
     for t in range(pos, L):
         lo = t // chunk * chunk if chunk else 0
         spots = [x for x in (lo, lo - 1, t, t - 1, lo + 1, (lo + t) // 2, lo + 63, lo + 64, lo + 16, 0) if 0 <= x <= t]
         for h in range(H):
-            if (t + h) % 3:
+            if lo and h == t % H:
+                q[t, h] = act.host(k[lo - 1, h // (H // G)])
+            elif (t + h) % 3:
                 s = spots[(t + 2 * h) % len(spots)]
                 q[t, h] = act.host(k[s, h // (H // G)] * (1 if (t + h) % 5 else -1))     # (or away from it: the sink takes over)
-                aims += s < lo
-    assert not chunk or pos < chunk or H < 2 or aims
     qn, kn = ho.rms(q.astype(F64), eps), ho.rms(k.astype(F64), eps)
     want = np.empty((T, H, V))
     for t in range(pos, L):
@@ -444,7 +443,7 @@ def check_far_token(lib, cfg, w, toks, far, matters, sizes_of, fine):
         e = Engine(m)
         for sizes in sizes_of(len(toks)):
             err = hm.row_errors(feed_portions(e, 0, toks, sizes), want)
-            assert np.max(err) < (fine if dtype == "float32" else LIMIT[dtype]), (dtype, sizes[:2], int(np.argmax(err)))
+            assert np.max(err) < (fine if dtype == "float32" else 0.15), (dtype, sizes[:2], int(np.argmax(err)))
         e.close()
         m.close()
 
