@@ -309,7 +309,7 @@ __device__ __forceinline__ float transposed_sum(float (&v)[32], int lane)
 
 // grid (heads, chunks), a thread per key (rounded up to whole warps); tokens t0 .. t1 - 1, those beyond count as zeros that
 // neither decay nor write.
-__global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* frags, float* updates, int t0, int t1)
+__global__ void __launch_bounds__(256, 2) k_delta_prepare(DeltaRule a, uint8_t* frags, float* updates, int t0, int t1)
 {
     extern __shared__ __align__(16) uint8_t sf[];     // the chunk's fragments
     __shared__ float s_part[8][256], s_norm[8][32];
@@ -323,16 +323,15 @@ __global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* fra
     pdl_wait();
     float k[kChunk], q[kChunk], g[kChunk];
     {
-        const bf16* pk = reinterpret_cast<const bf16*>(a.k) + gr * D + n;
-        const bf16* pq = reinterpret_cast<const bf16*>(a.q) + gr * D + n;
-        const float* pd = a.log_decay + (size_t)h * D + n;
+        const bf16* pk = reinterpret_cast<const bf16*>(a.k) + (size_t)first * a.ld + gr * D + n;
+        const bf16* pq = reinterpret_cast<const bf16*>(a.q) + (size_t)first * a.ld + gr * D + n;
+        const float* pd = a.log_decay + ((size_t)first * a.heads + h) * D + n;
+        const int left = key ? t1 - first : 0, step = a.heads * D;
 #pragma unroll
         for (int i = 0; i < kChunk; i++) {
-            const bool in = key && first + i < t1;
-            const size_t t = first + i;
-            k[i] = in ? act_load(pk + t * a.ld) : 0.0f;
-            q[i] = in ? act_load(pq + t * a.ld) : 0.0f;
-            g[i] = in ? pd[t * a.heads * D] : 0.0f;
+            k[i] = i < left ? act_load(pk + i * a.ld) : 0.0f;
+            q[i] = i < left ? act_load(pq + i * a.ld) : 0.0f;
+            g[i] = i < left ? pd[i * step] : 0.0f;
         }
     }
     if (tid < kChunk) s_beta[tid] = first + tid < t1 ? a.beta[(size_t)(first + tid) * a.heads + h] : 0.0f;
@@ -390,9 +389,11 @@ __global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* fra
         else { const int i = 16 - m + l - (32 - m); A[i * kChunk + 15 - m] = sum * s_beta[i]; }
     }
     __syncthreads();
-    auto entry = [](const float4 (&m)[kChunk][4], int i, int j) -> float {
-        const float4 x = m[i][j >> 2];
-        return (j & 3) == 0 ? x.x : (j & 3) == 1 ? x.y : (j & 3) == 2 ? x.z : x.w;
+    // the first n entries of a row
+    auto load_row = [](const float4 (&m)[kChunk][4], int i, int n, float (&r)[kChunk]) {
+#pragma unroll
+        for (int j = 0; j < 4; j++)
+            if (4 * j < n) *reinterpret_cast<float4*>(r + 4 * j) = m[i][j];
     };
     const size_t unit = (size_t)blockIdx.y * a.heads + h;
     if (key) {
@@ -420,13 +421,16 @@ __global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* fra
         for (int i = 0; i < kChunk; i++) {
             c *= g[i];
             float x = s_beta[i] * k[i] * c, y = q[i] * c;
+            alignas(16) float ar[kChunk], pr[kChunk];
+            load_row(sA, i, i, ar);
+            load_row(sP, i, i + 1, pr);
 #pragma unroll
             for (int j = 0; j < i; j++) {
-                x = fmaf(-entry(sA, i, j), w[j], x);
-                y = fmaf(-entry(sP, i, j), w[j], y);
+                x = fmaf(-ar[j], w[j], x);
+                y = fmaf(-pr[j], w[j], y);
             }
             w[i] = x;
-            z[i] = fmaf(-entry(sP, i, i), x, y);
+            z[i] = fmaf(-pr[i], x, y);
         }
         // keys n and n + 1 share a register: the even thread writes tokens 0 .. 7, the odd one 8 .. 15
         const unsigned live = D - (n & ~31) >= 32 ? 0xFFFFFFFFu : 0xFFFFu;
@@ -448,20 +452,24 @@ __global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* fra
     }
     float* up = updates + unit * update_floats(V);
     for (int p = tid; p < V; p += blockDim.x) {
-        const bf16* pv = reinterpret_cast<const bf16*>(a.v) + (size_t)h * V + p;
+        const bf16* pv = reinterpret_cast<const bf16*>(a.v) + (size_t)first * a.ld + (size_t)h * V + p;
+        const int left = t1 - first;
         float x[kChunk], u[kChunk], o[kChunk];
 #pragma unroll
-        for (int i = 0; i < kChunk; i++) x[i] = first + i < t1 ? act_load(pv + (size_t)(first + i) * a.ld) : 0.0f;
+        for (int i = 0; i < kChunk; i++) x[i] = i < left ? act_load(pv + i * a.ld) : 0.0f;
 #pragma unroll
         for (int i = 0; i < kChunk; i++) {
             float y = s_beta[i] * x[i], z = 0.0f;
+            alignas(16) float ar[kChunk], pr[kChunk];
+            load_row(sA, i, i, ar);
+            load_row(sP, i, i + 1, pr);
 #pragma unroll
             for (int j = 0; j < i; j++) {
-                y = fmaf(-entry(sA, i, j), u[j], y);
-                z = fmaf(entry(sP, i, j), u[j], z);
+                y = fmaf(-ar[j], u[j], y);
+                z = fmaf(pr[j], u[j], z);
             }
             u[i] = y;
-            o[i] = fmaf(entry(sP, i, i), y, z);
+            o[i] = fmaf(pr[i], y, z);
         }
         float* dst = up + (size_t)(p >> 4) * 512 + (p & 7) * 32 + ((p >> 3) & 1) * 2;
 #pragma unroll
@@ -477,6 +485,12 @@ __global__ void __launch_bounds__(256) k_delta_prepare(DeltaRule a, uint8_t* fra
     for (int i = tid; i < (int)(fragment_bytes(D) / 16); i += blockDim.x) dst[i] = reinterpret_cast<const uint4*>(sf)[i];
 }
 
+// (Not a barrier for the compiler: loads of other shared memory may pass it; an arrival on a barrier publishes it.)
+__device__ __forceinline__ void store_shared(uint32_t at, const uint32_t (&v)[4])
+{
+    asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(at), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]));
+}
+
 template <int NMAX>
 struct DeltaChunks {
     static constexpr int kStages = NMAX == 256 ? 3 : 4;
@@ -484,8 +498,9 @@ struct DeltaChunks {
     static size_t smem(int key_pad) { return kStages * fragment_bytes(key_pad) + 4 * kState; }
 };
 
-// grid (heads, value columns / 32): warps 0, 1 hold the state of 16 value columns each, warps 2, 3 read it out, warp 4 feeds.
-template <int NMAX>
+// grid (heads, value columns / 32): warps 0, 1 hold the state of 16 value columns each, warps 2, 3 read it out, warp 4 feeds.  kExact: the keys
+// are NMAX, so that no step of the products hangs on a branch.
+template <int NMAX, bool kExact>
 __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint8_t* frags, const float* updates, int t0, int t1, int chunks, int* err)
 {
     using S = DeltaChunks<NMAX>;
@@ -493,7 +508,7 @@ __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint
     extern __shared__ __align__(128) uint8_t smem[];
     __shared__ uint64_t full[S::kStages], empty[S::kStages], state_full[2][2], state_empty[2][2];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
-    const int h = blockIdx.x, D = a.key_pad, V = a.value_pad, ks_n = D / 16;
+    const int h = blockIdx.x, D = kExact ? NMAX : a.key_pad, V = a.value_pad, ks_n = D / 16;
     const int blocks = V / 16 - 2 * (int)blockIdx.y < 2 ? V / 16 - 2 * (int)blockIdx.y : 2;
     const uint32_t bytes = (uint32_t)fragment_bytes(D);
     uint8_t* s_state = smem + S::kStages * (size_t)bytes;
@@ -541,29 +556,35 @@ __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint
             if (!mbar_wait_bounded(&full[s], (uint32_t)(c / S::kStages) & 1u, err, 62)) break;
             if (c >= 2 && !mbar_wait_bounded(&state_empty[pair][b], (uint32_t)(c / 2 - 1) & 1u, err, 63)) break;
             const uint8_t* f = smem + s * (size_t)bytes;
+            const uint32_t to = smem_addr(mine + b * S::kState);
             float x[2][4] = {{u0.x, u0.y, u0.z, u0.w}, {u1.x, u1.y, u1.z, u1.w}}, y[2][4] = {}, z[2][4] = {};
             if (c + 1 < chunks) {
                 up += next_up;
                 u0 = *reinterpret_cast<const float4*>(up);
                 u1 = *reinterpret_cast<const float4*>(up + 4);
             }
+            const uint4* fw = reinterpret_cast<const uint4*>(f) + lane;
+            uint4 w0 = fw[0], w1 = fw[32];
 #pragma unroll
             for (int ks = 0; ks < KS; ks++) {
                 if (ks >= ks_n) break;
+                uint4 n0 = w0, n1 = w1;
+                if (ks + 1 < KS && ks + 1 < ks_n) { n0 = fw[(2 * ks + 2) * 32]; n1 = fw[(2 * ks + 3) * 32]; }
                 uint32_t ah[4], al[4];
                 split_bf16(st[2 * ks][0], st[2 * ks][1], ah[0], al[0]);
                 split_bf16(st[2 * ks][2], st[2 * ks][3], ah[1], al[1]);
                 split_bf16(st[2 * ks + 1][0], st[2 * ks + 1][1], ah[2], al[2]);
                 split_bf16(st[2 * ks + 1][2], st[2 * ks + 1][3], ah[3], al[3]);
-                *reinterpret_cast<uint4*>(mine + b * S::kState + ks * 1024) = make_uint4(ah[0], ah[1], ah[2], ah[3]);
-                *reinterpret_cast<uint4*>(mine + b * S::kState + ks * 1024 + 512) = make_uint4(al[0], al[1], al[2], al[3]);
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const uint4 w = *reinterpret_cast<const uint4*>(f + ((ks * 2 + e) * 32 + lane) * 16);
-                    mma_bf16(x[e], ah, w.x, w.y);
-                    mma_bf16(y[e], ah, w.z, w.w);
-                    mma_bf16(z[e], al, w.x, w.y);
-                }
+                store_shared(to + ks * 1024, ah);
+                store_shared(to + ks * 1024 + 512, al);
+                mma_bf16(x[0], ah, w0.x, w0.y);
+                mma_bf16(x[1], ah, w1.x, w1.y);
+                mma_bf16(y[0], ah, w0.z, w0.w);
+                mma_bf16(y[1], ah, w1.z, w1.w);
+                mma_bf16(z[0], al, w0.x, w0.y);
+                mma_bf16(z[1], al, w1.x, w1.y);
+                w0 = n0;
+                w1 = n1;
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(&state_full[pair][b]);
@@ -582,12 +603,17 @@ __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint
                 split_bf16(x[e][2] + (y[e][2] + z[e][2]), x[e][3] + (y[e][3] + z[e][3]), uh[2 * e + 1], ul[2 * e + 1]);
             }
 #pragma unroll
-            for (int j = 0; j < NT; j++) {
+            for (int j = 0; j < NT; j += 8) {
                 if (8 * j >= D) break;
-                const uint4 kf = *reinterpret_cast<const uint4*>(fk + (j * 32 + lane) * 16);
-                mma_bf16(st[j], uh, kf.x, kf.y);
-                mma_bf16(st[j], uh, kf.z, kf.w);
-                mma_bf16(st[j], ul, kf.x, kf.y);
+                uint4 kf[8];
+#pragma unroll
+                for (int i = 0; i < 8; i++) kf[i] = 8 * (j + i) < D ? *reinterpret_cast<const uint4*>(fk + ((j + i) * 32 + lane) * 16) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                for (int i = 0; i < 8; i++) mma_bf16(st[j + i], uh, kf[i].x, kf[i].y);
+#pragma unroll
+                for (int i = 0; i < 8; i++) mma_bf16(st[j + i], uh, kf[i].z, kf[i].w);
+#pragma unroll
+                for (int i = 0; i < 8; i++) mma_bf16(st[j + i], ul, kf[i].x, kf[i].y);
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(&empty[s]);
@@ -613,19 +639,28 @@ __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint
                 u0 = *reinterpret_cast<const float4*>(up);
                 u1 = *reinterpret_cast<const float4*>(up + 4);
             }
+            const uint4* fq = reinterpret_cast<const uint4*>(f) + lane;
+            const uint4* from = reinterpret_cast<const uint4*>(mine + b * S::kState);
+            uint4 hi = from[0], lo = from[32], w0 = fq[0], w1 = fq[32];
 #pragma unroll
             for (int ks = 0; ks < KS; ks++) {
                 if (ks >= ks_n) break;
-                const uint4 hi = *reinterpret_cast<const uint4*>(mine + b * S::kState + ks * 1024);
-                const uint4 lo = *reinterpret_cast<const uint4*>(mine + b * S::kState + ks * 1024 + 512);
                 const uint32_t ah[4] = {hi.x, hi.y, hi.z, hi.w}, al[4] = {lo.x, lo.y, lo.z, lo.w};
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const uint4 w = *reinterpret_cast<const uint4*>(f + ((ks * 2 + e) * 32 + lane) * 16);
-                    mma_bf16(x[e], ah, w.x, w.y);
-                    mma_bf16(y[e], ah, w.z, w.w);
-                    mma_bf16(z[e], al, w.x, w.y);
+                uint4 n0 = w0, n1 = w1;
+                if (ks + 1 < KS && ks + 1 < ks_n) {
+                    n0 = fq[(2 * ks + 2) * 32];
+                    n1 = fq[(2 * ks + 3) * 32];
+                    hi = from[(2 * ks + 2) * 32];
+                    lo = from[(2 * ks + 3) * 32];
                 }
+                mma_bf16(x[0], ah, w0.x, w0.y);
+                mma_bf16(x[1], ah, w1.x, w1.y);
+                mma_bf16(y[0], ah, w0.z, w0.w);
+                mma_bf16(y[1], ah, w1.z, w1.w);
+                mma_bf16(z[0], al, w0.x, w0.y);
+                mma_bf16(z[1], al, w1.x, w1.y);
+                w0 = n0;
+                w1 = n1;
             }
             __syncwarp();
             if (lane == 0) { mbar_arrive(&state_empty[pair][b]); mbar_arrive(&empty[s]); }
@@ -645,10 +680,10 @@ __global__ void __launch_bounds__(160, 1) k_delta_chunks(DeltaRule a, const uint
     }
 }
 
-template <int NMAX>
+template <int NMAX, bool kExact>
 static int launch_chunks(const DeltaRule& a, int T, cudaStream_t s)
 {
-    int rc = allow_smem<k_delta_chunks<NMAX>>((int)DeltaChunks<NMAX>::smem(NMAX));
+    int rc = allow_smem<k_delta_chunks<NMAX, kExact>>((int)DeltaChunks<NMAX>::smem(NMAX));
     if (rc) return rc;
     if ((rc = allow_smem<k_delta_prepare>((int)fragment_bytes(256)))) return rc;
     for (int t0 = 0; t0 < T; t0 += kSegmentChunks * kChunk) {
@@ -657,7 +692,7 @@ static int launch_chunks(const DeltaRule& a, int T, cudaStream_t s)
         float* updates = (float*)(frags + (size_t)chunks * a.heads * fragment_bytes(a.key_pad));
         if ((rc = launch_ordered(k_delta_prepare, dim3(a.heads, chunks), (a.key_pad + 31) / 32 * 32, fragment_bytes(a.key_pad), s, a, frags, updates, t0, t1)))
             return rc;
-        if ((rc = launch_ordered(k_delta_chunks<NMAX>, dim3(a.heads, (a.value_pad + 31) / 32), 160, DeltaChunks<NMAX>::smem(a.key_pad), s, a,
+        if ((rc = launch_ordered(k_delta_chunks<NMAX, kExact>, dim3(a.heads, (a.value_pad + 31) / 32), 160, DeltaChunks<NMAX>::smem(a.key_pad), s, a,
                                  (const uint8_t*)frags, (const float*)updates, t0, t1, chunks, device_error_flag())))
             return rc;
     }
@@ -684,9 +719,11 @@ int delta_rule(const DeltaRule& a, int T, bool act_bf16, cudaStream_t s)
     if (a.norm_w && (T > 1 || !a.gate || !delta_token_norms(a.key_pad, a.value_pad))) return latch(BPDQ_ERR_ARG);
     if (T == 1) return act_bf16 ? delta_token<bf16>(a, s) : delta_token<float>(a, s);
     if (a.scratch && takes_chunks(a.key_pad, T, act_bf16)) {
-        if (a.key_pad <= 64) return launch_chunks<64>(a, T, s);
-        if (a.key_pad <= 128) return launch_chunks<128>(a, T, s);
-        return launch_chunks<256>(a, T, s);
+        if (a.key_pad == 64) return launch_chunks<64, true>(a, T, s);
+        if (a.key_pad == 128) return launch_chunks<128, true>(a, T, s);
+        if (a.key_pad < 64) return launch_chunks<64, false>(a, T, s);
+        if (a.key_pad < 128) return launch_chunks<128, false>(a, T, s);
+        return launch_chunks<256, false>(a, T, s);
     }
     return act_bf16 ? delta_recurrence<bf16>(a, T, s) : delta_recurrence<float>(a, T, s);
 }

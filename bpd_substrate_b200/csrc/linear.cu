@@ -325,7 +325,10 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
             if (l.mode == kLinResidual && live) {
                 pw = post.w[n]; pb = post.b[n];
                 if (next.w) { nw = next.w[n]; nb = next.b[n]; }
+            } else if (l.mode == kLinLogDecay && live) {
+                pw = l.neg_exp_a[n]; pb = l.dt_bias[n];
             }
+            const bool plain_f32 = l.mode == kLinF32 && l.cap == 0.0f;
             // rows of this warp that are only rounded and stored (after a GELU)
             const int n_end = (n - lane) + 32;
             const bool plain_warp = !((l.N | l.ld_out) & 1) &&
@@ -373,6 +376,14 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
                         const int t = t0 + j + (lane & 1);
                         if (live && t < T) *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf16*>(l.out) + (size_t)t * l.ld_out + (n & ~1)) = two;
                     }
+                } else if (plain_f32) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (live && t0 + j < T) reinterpret_cast<float*>(l.out)[(size_t)(t0 + j) * l.ld_out + n] = __int_as_float(v[j]);
+                } else if (l.mode == kLinLogDecay) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (live && t0 + j < T) l.dt[(size_t)(t0 + j) * l.ld_dt + n] = pw * softplus_act<bf16>(__int_as_float(v[j]) + pb);
                 } else if (live) {
 #pragma unroll
                     for (int j = 0; j < 16; j++)
