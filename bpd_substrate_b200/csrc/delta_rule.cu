@@ -309,7 +309,8 @@ __device__ __forceinline__ float transposed_sum(float (&v)[32], int lane)
 
 // grid (heads, chunks), a thread per key (rounded up to whole warps); tokens t0 .. t1 - 1, those beyond count as zeros that
 // neither decay nor write.
-__global__ void __launch_bounds__(256, 2) k_delta_prepare(DeltaRule a, uint8_t* frags, float* updates, int t0, int t1)
+template <int kThreads, int kBlocks>
+__global__ void __launch_bounds__(kThreads, kBlocks) k_delta_prepare(DeltaRule a, uint8_t* frags, float* updates, int t0, int t1)
 {
     extern __shared__ __align__(16) uint8_t sf[];     // the chunk's fragments
     __shared__ float s_part[8][256], s_norm[8][32];
@@ -685,12 +686,13 @@ static int launch_chunks(const DeltaRule& a, int T, cudaStream_t s)
 {
     int rc = allow_smem<k_delta_chunks<NMAX, kExact>>((int)DeltaChunks<NMAX>::smem(NMAX));
     if (rc) return rc;
-    if ((rc = allow_smem<k_delta_prepare>((int)fragment_bytes(256)))) return rc;
+    constexpr auto prepare = k_delta_prepare<NMAX == 256 ? 256 : 128, NMAX == 256 ? 1 : 3>;
+    if ((rc = allow_smem<prepare>((int)fragment_bytes(256)))) return rc;
     for (int t0 = 0; t0 < T; t0 += kSegmentChunks * kChunk) {
         const int t1 = T - t0 < kSegmentChunks * kChunk ? T : t0 + kSegmentChunks * kChunk, chunks = (t1 - t0 + kChunk - 1) / kChunk;
         uint8_t* frags = (uint8_t*)a.scratch;
         float* updates = (float*)(frags + (size_t)chunks * a.heads * fragment_bytes(a.key_pad));
-        if ((rc = launch_ordered(k_delta_prepare, dim3(a.heads, chunks), (a.key_pad + 31) / 32 * 32, fragment_bytes(a.key_pad), s, a, frags, updates, t0, t1)))
+        if ((rc = launch_ordered(prepare, dim3(a.heads, chunks), (a.key_pad + 31) / 32 * 32, fragment_bytes(a.key_pad), s, a, frags, updates, t0, t1)))
             return rc;
         if ((rc = launch_ordered(k_delta_chunks<NMAX, kExact>, dim3(a.heads, (a.value_pad + 31) / 32), 160, DeltaChunks<NMAX>::smem(a.key_pad), s, a,
                                  (const uint8_t*)frags, (const float*)updates, t0, t1, chunks, device_error_flag())))

@@ -77,8 +77,10 @@ struct ScoreMap {
     __device__ __forceinline__ float operator()(float s) const
     {
         if (in == 0.0f) return s * plain;
-        return fmaf(-2.0f * out, __fdividef(1.0f, 1.0f + ex2(s * in)), out);
+        return fmaf(-2.0f * out, below(s), out);
     }
+    // (1 - tanh) / 2 of a capped score
+    __device__ __forceinline__ float below(float s) const { return __fdividef(1.0f, 1.0f + ex2(s * in)); }
 };
 
 // ------------------------------------------------------------------ few queries, bf16
@@ -283,8 +285,12 @@ static size_t tile_smem(int dim_pad, int dv)
     return (size_t)(kTileRows + 2 * kKeyBlock) * (dim_pad + 8) * 2 + 2 * (size_t)kKeyBlock * (dv + 8) * 2;
 }
 
+// A capped score cannot exceed the cap, so weights can be taken relative to it and no maximum is tracked.  With a sink the sum is
+// at least e^-cap; up to this cap whatever underflows beside that is below fp32's resolution.
+constexpr float kBoundedCap = 64.0f;
+
 // grid (row tiles, groups, value slices of DV); four warps of 16 rows.
-template <int DV>
+template <int DV, bool kBounded>
 __global__ void __launch_bounds__(128) k_grouped_tile_mma(GroupedShape p, const bf16* u, int ld_u, const bf16* cache, bf16* o, const int* pos_p, int T)
 {
     constexpr int LDV = DV + 8;
@@ -342,7 +348,7 @@ __global__ void __launch_bounds__(128) k_grouped_tile_mma(GroupedShape p, const 
     const ScoreMap score(p);
     float mx[2], sum[2];
     mx[0] = mx[1] = p.sink ? 0.0f : -INFINITY;
-    sum[0] = sum[1] = (p.sink && t4 == 0) ? 1.0f : 0.0f;        // (a row's four lanes are added up at the end)
+    sum[0] = sum[1] = (p.sink && t4 == 0) ? (kBounded ? ex2(-score.out) : 1.0f) : 0.0f;        // (a row's four lanes are added up at the end)
     int b = 0;
     for (int k0 = k_begin; k0 < k_end; k0 += kKeyBlock, b ^= 1) {
         cp_async_wait_all();
@@ -363,6 +369,24 @@ __global__ void __launch_bounds__(128) k_grouped_tile_mma(GroupedShape p, const 
         const bool edge = k0 + kKeyBlock - 1 > w_last || k0 < w_lo;
 #pragma unroll
         for (int e = 0; e < 2; e++) {
+            if (kBounded) {
+                const float f = -2.0f * score.out;
+                float w = 0.0f;
+#pragma unroll
+                for (int n = 0; n < 8; n++)
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        float v = ex2(f * score.below(s[n][2 * e + c]));
+                        if (edge) {
+                            const int k = k0 + 8 * n + 2 * t4 + c;
+                            if (k > last[e] || k < lo[e]) v = 0.0f;
+                        }
+                        s[n][2 * e + c] = v;
+                        w += v;
+                    }
+                sum[e] += w;
+                continue;
+            }
             float m = mx[e];
 #pragma unroll
             for (int n = 0; n < 8; n++)
@@ -535,13 +559,13 @@ static int launch_split(const GroupedShape& p, const bf16* u, int ld_u, const bf
                           ld_u, cache, o, pos, T);
 }
 
-template <int DV>
+template <int DV, bool kBounded>
 static int launch_tile(const GroupedShape& p, const bf16* u, int ld_u, const bf16* cache, bf16* o, const int* pos, int T, cudaStream_t s)
 {
-    int rc = allow_smem<k_grouped_tile_mma<DV>>(220 * 1024);
+    int rc = allow_smem<k_grouped_tile_mma<DV, kBounded>>(220 * 1024);
     if (rc) return rc;
     const dim3 grid((unsigned)(((long)T * p.share() + kTileRows - 1) / kTileRows), p.groups, (p.value_pad + DV - 1) / DV);
-    return launch_ordered(k_grouped_tile_mma<DV>, grid, 128, tile_smem(p.dim_pad, DV), s, p, u, ld_u, cache, o, pos, T);
+    return launch_ordered(k_grouped_tile_mma<DV, kBounded>, grid, 128, tile_smem(p.dim_pad, DV), s, p, u, ld_u, cache, o, pos, T);
 }
 
 int grouped_attention(const GroupedShape& p, const void* u, int ld_u, const void* cache, void* o, const int* pos, int T, bool act_bf16,
@@ -556,8 +580,11 @@ int grouped_attention(const GroupedShape& p, const void* u, int ld_u, const void
         if (most <= 128) return launch_split<4, 2>(p, q, ld_u, c, out, pos, T, s);
         return launch_split<8, 4>(p, q, ld_u, c, out, pos, T, s);
     }
-    if (tile_smem(p.dim_pad, p.value_pad <= 64 ? 64 : 128) <= 220 * 1024)
-        return p.value_pad <= 64 ? launch_tile<64>(p, q, ld_u, c, out, pos, T, s) : launch_tile<128>(p, q, ld_u, c, out, pos, T, s);
+    if (tile_smem(p.dim_pad, p.value_pad <= 64 ? 64 : 128) <= 220 * 1024) {
+        const bool bounded = p.sink && p.cap > 0.0f && p.cap <= kBoundedCap;
+        if (p.value_pad <= 64) return bounded ? launch_tile<64, true>(p, q, ld_u, c, out, pos, T, s) : launch_tile<64, false>(p, q, ld_u, c, out, pos, T, s);
+        return bounded ? launch_tile<128, true>(p, q, ld_u, c, out, pos, T, s) : launch_tile<128, false>(p, q, ld_u, c, out, pos, T, s);
+    }
     return launch_rows<bf16>(p, u, ld_u, cache, o, pos, T, s);
 }
 

@@ -251,6 +251,13 @@ def test_grouped_attention_rows_used_again(lib, bf16, T, pos, chunk, rows):
 
 
 @pytest.mark.parametrize("bf16", ACTS)
+@pytest.mark.parametrize("cap", [2.0, 60.0, 90.0, 500.0])
+def test_grouped_attention_caps(lib, bf16, cap):
+    for T, pos in ((1, 70), (90, 20)):
+        attention_case(lib, bf16, T, pos, 4, 2, 32, 72, 48, cap=cap)
+
+
+@pytest.mark.parametrize("bf16", ACTS)
 @pytest.mark.parametrize("T,pos", [(1, 130), (90, 20)])
 def test_grouped_attention_without_sink_or_cap(lib, bf16, T, pos):
     attention_case(lib, bf16, T, pos, 4, 2, 32, 32, 48, sink=0)
