@@ -250,6 +250,7 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
     pdl_launch_dependents();
 
     const int n_tiles = (l.N + S::kRows - 1) / S::kRows, t_tiles = (T + BN - 1) / BN;
+    // tokens vary fastest: the CTAs at work share few rows of weights, which go through HBM once
     const int tiles = n_tiles * t_tiles, kb_n = (l.K + S::kDepth - 1) / S::kDepth;
 
     if (warp == 0) {
@@ -260,11 +261,11 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
             auto weights = [&](long i, int s) {
                 const int tile = blockIdx.x + (int)(i / kb_n) * gridDim.x, kb = (int)(i % kb_n);
                 mbar_expect_tx(&full[s], S::kStageBytes);
-                tma_rows_2d(ring + (size_t)s * S::kStageBytes, &wmap, kb * S::kDepth, (tile % n_tiles) * S::kRows, &full[s]);
+                tma_rows_2d(ring + (size_t)s * S::kStageBytes, &wmap, kb * S::kDepth, (tile / t_tiles) * S::kRows, &full[s]);
             };
             auto tokens = [&](long i, int s) {
                 const int tile = blockIdx.x + (int)(i / kb_n) * gridDim.x, kb = (int)(i % kb_n);
-                tma_rows_2d(ring + (size_t)s * S::kStageBytes + S::kABytes, &xmap, kb * S::kDepth, (tile / n_tiles) * BN, &full[s]);
+                tma_rows_2d(ring + (size_t)s * S::kStageBytes + S::kABytes, &xmap, kb * S::kDepth, (tile % t_tiles) * BN, &full[s]);
             };
             const long ahead = steps < kStages ? steps : kStages;
             for (long i = 0; i < ahead; i++) weights(i, (int)i);
@@ -316,8 +317,8 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
             const int a = local & 1;
             if (!mbar_wait_bounded(&acc_full[a], (uint32_t)(local >> 1) & 1u, err, 44)) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const int n = (tile % n_tiles) * S::kRows + r;
-            const int tb = (tile / n_tiles) * BN + half * kCols;
+            const int n = (tile / t_tiles) * S::kRows + r;
+            const int tb = (tile % t_tiles) * BN + half * kCols;
             const bool live = n < l.N;
             const uint32_t ta = tmem_base + ((uint32_t)(32 * quarter) << 16) + (uint32_t)(a * BN + half * kCols);
             DynTanh post = l.post, next = l.next;
@@ -328,6 +329,8 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
             } else if (l.mode == kLinLogDecay && live) {
                 pw = l.neg_exp_a[n]; pb = l.dt_bias[n];
             }
+            const bool is_step = l.mode == kLinMixerIn && live && n >= l.dt_row;      // (lanes of one warp may differ)
+            if (is_step && l.dt_bias) pb = l.dt_bias[n - l.dt_row];
             const bool plain_f32 = l.mode == kLinF32 && l.cap == 0.0f;
             // rows of this warp that are only rounded and stored (after a GELU)
             const int n_end = (n - lane) + 32;
@@ -384,6 +387,13 @@ k_linear_tc5(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ C
 #pragma unroll
                     for (int j = 0; j < 16; j++)
                         if (live && t0 + j < T) l.dt[(size_t)(t0 + j) * l.ld_dt + n] = pw * softplus_act<bf16>(__int_as_float(v[j]) + pb);
+                } else if (is_step) {
+                    float q[16];
+#pragma unroll
+                    for (int j = 0; j < 16; j++) q[j] = l.dt_bias ? softplus_act<bf16>(__int_as_float(v[j]) + pb) : sigmoid_act<bf16>(__int_as_float(v[j]));
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (t0 + j < T) l.dt[(size_t)(t0 + j) * l.ld_dt + n - l.dt_row] = q[j];
                 } else if (live) {
 #pragma unroll
                     for (int j = 0; j < 16; j++)
