@@ -18,6 +18,10 @@ def _number(where, d, key, positive=False):
     return float(v)
 
 
+def _chunk(m):
+    return m["mask"]["size"] if m.get("mask") is not None else 0
+
+
 class VuzelixSpec(DecoderSpec):
     architecture = "Vuzelix"
     portion = 4096          # attention layers keep this many rows beyond a chunk: a step of as many tokens overwrites none it needs
@@ -44,7 +48,8 @@ class VuzelixSpec(DecoderSpec):
             else:
                 _number(where, m, "scale")
                 _number(where, m, "softcap", True)
-                _positive(where, m.get("mask") or {}, "size")
+                if m.get("mask") is not None:       # without one a position sees everything before it
+                    _positive(where, m["mask"], "size")
                 j = m.get("kv_from")
                 if j is not None:
                     own = self.layers[j] if isinstance(j, int) and 0 <= j < i else None
@@ -98,9 +103,9 @@ class VuzelixSpec(DecoderSpec):
                 parts.append(StatePart(f"l{i}.state", 4 * m["heads"] * D * V))
                 parts.append(StatePart(f"l{i}.tail", 4 * max(1, m["conv"] - 1) * (2 * m["kv_heads"] * D + m["heads"] * V)))
             elif m.get("kv_from") is None:
-                reach = max(u["mixer"]["mask"]["size"] for j, u in enumerate(self.layers)
-                            if u["type"] == "attention" and i in (j, u["mixer"].get("kv_from")))
-                parts.append(StatePart(f"l{i}.cache", a * m["kv_heads"] * (D + V), rows=True, zero=False, limit=reach + self.portion))
+                reach = [_chunk(u["mixer"]) for j, u in enumerate(self.layers) if u["type"] == "attention" and i in (j, u["mixer"].get("kv_from"))]
+                parts.append(StatePart(f"l{i}.cache", a * m["kv_heads"] * (D + V), rows=True, zero=False,
+                                       limit=max(reach) + self.portion if all(reach) else 0))
         return parts
 
     def pack_layer(self, i, get):
@@ -124,7 +129,7 @@ class VuzelixSpec(DecoderSpec):
             else:
                 out.ints["kv_from"] = m["kv_from"]
             out.mats["w_in"] = np.concatenate(w_in)
-            out.ints["chunk"] = m["mask"]["size"]
+            out.ints["chunk"] = _chunk(m)
             out.floats.update(scale=float(m["scale"]), softcap=float(m["softcap"]))
         else:
             a, g = self.ranks[i]

@@ -103,7 +103,7 @@ def attention(m, w, p, h, pos, st, eps):
     """st: the cache of the layer whose keys are used; its newest entry is this token's."""
     H, G = m["heads"], m["kv_heads"]
     q = rms((w[p + ".q"] @ h).reshape(H, m["dim"]), eps)
-    seen = [j for j in range(pos + 1) if sees(pos, j, m["mask"]["size"])]
+    seen = [j for j in range(pos + 1) if sees(pos, j, m["mask"]["size"] if m.get("mask") else 0)]
     o = []
     for n in range(H):
         g = n // (H // G)

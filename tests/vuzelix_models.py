@@ -10,7 +10,9 @@ def delta(heads, kv_heads, dim, vdim, conv):
 
 
 def attention(heads, kv_heads, dim, vdim, chunk, scale, softcap, kv_from=None):
-    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk}, "scale": scale, "softcap": softcap}
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "softcap": softcap}
+    if chunk:
+        m["mask"] = {"size": chunk}
     if kv_from is not None:
         m["kv_from"] = kv_from
     return m
@@ -26,7 +28,7 @@ def config(vocab, width, streams, layers, eps=1e-5, embed=3.0, mult=0.6, cap=12.
 
 
 # both mixers with and without a feed-forward; shared key heads, other chunks than the owner of the keys, value sizes above and below
-# key sizes, sizes that are no multiples of anything; no convolution window; one stream and the most streams
+# key sizes, sizes that are no multiples of anything; no convolution window, no chunks; one stream and the most streams
 CONFIGS = {
     "mixed": config(211, 72, 2, [
         layer("channel_delta", delta(6, 2, 24, 40, 4), 88),
@@ -50,6 +52,7 @@ CONFIGS = {
         layer("channel_delta", delta(2, 2, 136, 264, 3), 40),
         layer("attention", attention(2, 1, 120, 200, 90, 0.2, 20.0), 40),
         layer("attention", attention(3, 1, 264, 24, 33, 0.15, 8.0)),
+        layer("attention", attention(2, 2, 16, 32, 0, 0.6, 8.0)),
         layer("channel_delta", delta(2, 1, 264, 16, 4), 30),
     ]),
 }
